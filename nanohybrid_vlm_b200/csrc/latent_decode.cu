@@ -5,7 +5,7 @@
 // beforehand) and the result is a weighted sum of latents per head, [rank], which the caller expands into values.
 //
 // The heads of one token are the 16 rows of an mma tile, so the keys of a request are read once for up to 16 heads.
-// The keys a token sees are cut into `n_splits` runs of whole tiles of 64 keys; block (split, token, group of 16
+// The keys a token sees (all up to itself, or with a window the last `window` of them) are cut into `n_splits` runs of whole tiles of 64 keys; block (split, token, group of 16
 // heads) writes an unnormalised partial sum with its running maximum and denominator, and a second kernel merges the
 // partial sums of a token and head, where the sink (exp(sink) in the denominator, once) joins.  The cutting depends
 // on the token's position and on `n_splits` only.
@@ -58,7 +58,7 @@ template <int NT>
 __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(
     float* __restrict__ part_o, float* __restrict__ part_ml, const bf16* __restrict__ q, int q_stride,
     const bf16* __restrict__ pages, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ cu_q,
-    const int* __restrict__ kv_len, int n_seqs, int H, int rank, int row, int page_size, int n_pages, float scale) {
+    const int* __restrict__ kv_len, int n_seqs, int H, int rank, int row, int page_size, int n_pages, float scale, int window) {
   extern __shared__ __align__(16) unsigned char ld_smem[];
   pdl_prologue();
   const int split = blockIdx.x, n_splits = gridDim.x, tok = blockIdx.y, h0 = blockIdx.z * 16;
@@ -74,10 +74,11 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(
   // the request of this token and the token's position
   int seq = 0;
   while (seq + 1 < n_seqs && cu_q[seq + 1] <= tok) ++seq;
-  const int pos = kv_len[seq] - (cu_q[seq + 1] - tok);  // it sees keys 0 .. pos
-  const int tiles_total = pos / LD_BN + 1;
+  const int pos = kv_len[seq] - (cu_q[seq + 1] - tok);  // it sees keys lo .. pos
+  const int lo = nhv_first_key(pos, window, 0);
+  const int tile_lo = lo / LD_BN, tiles_total = pos / LD_BN + 1 - tile_lo;
   const int per = (tiles_total + n_splits - 1) / n_splits;
-  const int tile0 = split * per, tile1 = min(tile0 + per, tiles_total);
+  const int tile0 = tile_lo + split * per, tile1 = min(tile0 + per, tile_lo + tiles_total);
   const size_t part = ((size_t)tok * H) * n_splits + split;     // + h * n_splits
   if (tile0 >= tile1 || pos < 0) {                      // nothing for this block: a partial sum that weighs nothing
     for (int r = tid; r < 16 && h0 + r < H; r += LD_THREADS) {
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(
     int mine = -1;                                      // lane i looks up the page of key warp + 16 i
     {
       const int j = tile * LD_BN + warp + LD_WARPS * (lane % (LD_BN / LD_WARPS));
-      if (j <= pos) mine = table[j / page_size];
+      if (j >= lo && j <= pos) mine = table[j / page_size];
     }
 #pragma unroll
     for (int i = 0; i < LD_BN / LD_WARPS; ++i) {
@@ -169,7 +170,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int j = tile * LD_BN + kg * 8 + 2 * t4 + (e & 1);
-        s[e] = j <= pos ? s[e] * sc2 : -INFINITY;
+        s[e] = j >= lo && j <= pos ? s[e] * sc2 : -INFINITY;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[e]);
       }
     }
@@ -304,7 +305,7 @@ NHV_API int nhv_latent_decode_supports(int H, int rank, int row) {
 // q_stride apart; out: [T, H, rank] with rows out_stride apart.
 NHV_API int nhv_latent_decode(void* out, int out_stride, const void* q, int q_stride, const void* pages,
                               const int* block_table, int bt_stride, const int* cu_q, const int* kv_len, int n_seqs,
-                              int n_tokens, int H, int rank, int row, int page_size, int n_pages, float scale,
+                              int n_tokens, int H, int rank, int row, int page_size, int n_pages, float scale, int window,
                               const float* sinks, int n_splits, float* part_o, float* part_ml, cudaStream_t stream) {
   if (n_tokens == 0 || n_seqs == 0) return 0;
   NHV_REQUIRE(nhv_latent_decode_supports(H, rank, row), "latent_decode: %d heads, a latent of %d in rows of %d: not taken", H, rank, row);
@@ -320,7 +321,7 @@ NHV_API int nhv_latent_decode(void* out, int out_stride, const void* q, int q_st
                "latent_decode");                                                                                     \
     nhv_launch(latent_decode_kernel<NT>, grid, LD_THREADS, smem, stream, part_o, part_ml, (const bf16*)q, q_stride,  \
                (const bf16*)pages, block_table, bt_stride, cu_q, kv_len, n_seqs, H, rank, row, page_size, n_pages,   \
-               scale);                                                                                               \
+               scale, window);                                                                                               \
   } while (0)
   const int ntw = (((rank >> 3) + LD_WARPS - 1) / LD_WARPS + 1) & ~1;
   if (ntw <= 2) LAUNCH(2);

@@ -3,8 +3,9 @@
 // many tokens that costs far fewer operations than attending over the latents themselves, whose rows are several
 // times a head's size).
 //
-// Temporary rows: request s owns rows [row0[s], row0[s] + 64 * ceil(kv_len[s] / 64)), row0 a multiple of 64, so that
-// 64 rows are one temporary page.
+// Temporary rows: request s owns a run of rows from row0[s] on, a multiple of 64, so that 64 rows are one temporary page;
+// they hold its tokens from first[s] (a multiple of 64) to its last: first is 0, or where a window is in force the tile of
+// the first key that one of the step's tokens sees.
 //
 // latent_gather:    cache pages with one plane ([page][1][1][slot][row]: latent [rank], rotated key part [dr]) ->
 //                   lat [rows, rank] and kr [rows, dr], contiguous; rows past a request's last token are cleared, so
@@ -20,15 +21,16 @@ constexpr int LE_TILE = 64;     // rows of a temporary page
 template <typename T>
 __global__ void latent_gather_kernel(T* __restrict__ lat, T* __restrict__ kr, const T* __restrict__ pages,
                                      const int* __restrict__ block_table, int bt_stride, const int* __restrict__ kv_len,
-                                     const int* __restrict__ row0, int rank, int dr, int row, int page_size, int n_pages) {
+                                     const int* __restrict__ row0, const int* __restrict__ first, int rank, int dr, int row,
+                                     int page_size, int n_pages) {
   pdl_prologue();
   const int s = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int total = kv_len[s];
   const int padded = (total + LE_TILE - 1) / LE_TILE * LE_TILE;
-  const int j = blockIdx.x * (blockDim.x >> 5) + warp;
+  const int i = blockIdx.x * (blockDim.x >> 5) + warp, j = first[s] + i;
   if (j >= padded) return;
-  const size_t r = (size_t)row0[s] + j;
+  const size_t r = (size_t)row0[s] + i;
   const T* src = nullptr;
   if (j < total) {
     const int page = block_table[(size_t)s * bt_stride + j / page_size];
@@ -75,17 +77,17 @@ __global__ void latent_assemble_kernel(T* __restrict__ tmp, T* __restrict__ qp, 
 }
 
 NHV_API int nhv_latent_gather(int dtype, void* lat, void* kr, const void* pages, const int* block_table, int bt_stride,
-                              const int* kv_len, const int* row0, int n_seqs, int max_kv_len, int rank, int dr, int row,
+                              const int* kv_len, const int* row0, const int* first, int n_seqs, int max_rows, int rank, int dr, int row,
                               int page_size, int n_pages, cudaStream_t stream) {
-  if (n_seqs == 0 || max_kv_len == 0) return 0;
+  if (n_seqs == 0 || max_rows == 0) return 0;
   NHV_REQUIRE(rank > 0 && dr >= 0 && row >= rank + dr && page_size > 0 && n_pages > 0 && bt_stride > 0,
               "latent_gather: bad sizes");
   const int warps = 8;
-  const int padded = (max_kv_len + LE_TILE - 1) / LE_TILE * LE_TILE;
+  const int padded = (max_rows + LE_TILE - 1) / LE_TILE * LE_TILE;
   dim3 grid((padded + warps - 1) / warps, n_seqs);
 #define LAUNCH(T)                                                                                                       \
   nhv_launch(latent_gather_kernel<T>, grid, warps * 32, 0, stream, (T*)lat, (T*)kr, (const T*)pages, block_table,        \
-             bt_stride, kv_len, row0, rank, dr, row, page_size, n_pages)
+             bt_stride, kv_len, row0, first, rank, dr, row, page_size, n_pages)
   if (dtype == NHV_F32) LAUNCH(float);
   else if (dtype == NHV_BF16) LAUNCH(__nv_bfloat16);
   else NHV_REQUIRE(false, "latent_gather: unknown dtype %d", dtype);

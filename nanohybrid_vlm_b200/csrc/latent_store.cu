@@ -4,7 +4,7 @@
 // One warp per (token, item).  Item 0 takes the token's row kv [rank + dr] of the down projection: the first `rank`
 // elements are divided by their root mean square (eps inside the root) and multiplied by a weight [rank]: the latent;
 // the last dr elements are one key part shared by all heads, of which the first rotary_dim rotate (element i with
-// i + rotary_dim / 2, angles from the table).  Both go to the token's slot of a page with one plane,
+// i + rotary_dim / 2, or (interleaved) element 2i with 2i + 1; angles from the table).  Both go to the token's slot of a page with one plane,
 // [page][1][1][slot_in_page][row], row >= rank + dr, latent first; the rest of the row is cleared.
 // Items 1 .. H take head h of q [T, H, dn + dr]: its last dr elements, rotated the same way, go to
 // q_lat [T, H, rank + dr] behind the `rank` elements that a product with the keys' expansion fills.
@@ -20,7 +20,7 @@ __global__ void latent_rope_store_kernel(const T* __restrict__ kv, int kv_stride
                                          const int* __restrict__ slot_mapping, const int* __restrict__ positions,
                                          const float* __restrict__ cos_sin, int rotary_dim, int max_position,
                                          int n_tokens, int H, int dn, int dr, int rank, int row, int page_size,
-                                         int n_pages, float eps, const T* __restrict__ weight) {
+                                         int n_pages, float eps, const T* __restrict__ weight, int interleaved) {
   extern __shared__ float smem[];
   pdl_prologue();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -37,6 +37,10 @@ __global__ void latent_rope_store_kernel(const T* __restrict__ kv, int kv_stride
     cs = cos_sin + (size_t)pos * rotary_dim;                    // cos[0..half) then sin[0..half)
   }
   auto turned = [&](const float* x, int c) {                    // element c of the rotated part x [dr]
+    if (cs && interleaved && c < rotary_dim) {
+      const int i = c >> 1;                                     // the pair (2i, 2i + 1) turns by angle i
+      return (c & 1) ? x[c] * cs[i] + x[c - 1] * cs[half + i] : x[c] * cs[i] - x[c + 1] * cs[half + i];
+    }
     if (cs && c < half) return x[c] * cs[c] - x[c + half] * cs[half + c];
     if (cs && c < rotary_dim) return x[c] * cs[c - half] + x[c - half] * cs[c];
     return x[c];
@@ -70,7 +74,7 @@ NHV_API int nhv_latent_rope_store(int dtype, const void* kv, int kv_stride, cons
                                   int q_lat_stride, void* pages, const int* slot_mapping, const int* positions,
                                   const float* cos_sin, int rotary_dim, int max_position, int n_tokens, int H, int dn,
                                   int dr, int rank, int row, int page_size, int n_pages, float eps, const void* weight,
-                                  cudaStream_t stream) {
+                                  int interleaved, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   NHV_REQUIRE(n_tokens > 0 && H > 0 && dn >= 0 && dr >= 0 && rank > 0, "latent_rope_store: bad sizes");
   NHV_REQUIRE(rank + dr <= LS_MAX_ROW, "latent_rope_store: a row of %d elements is beyond the supported %d", rank + dr, LS_MAX_ROW);
@@ -84,7 +88,7 @@ NHV_API int nhv_latent_rope_store(int dtype, const void* kv, int kv_stride, cons
 #define LAUNCH(T)                                                                                                   \
   nhv_launch(latent_rope_store_kernel<T>, blocks, LS_WARPS * 32, smem, stream, (const T*)kv, kv_stride, (const T*)q, \
              q_stride, (T*)q_lat, q_lat_stride, (T*)pages, slot_mapping, positions, cos_sin, rotary_dim,            \
-             max_position, n_tokens, H, dn, dr, rank, row, page_size, n_pages, eps, (const T*)weight)
+             max_position, n_tokens, H, dn, dr, rank, row, page_size, n_pages, eps, (const T*)weight, interleaved)
   if (dtype == NHV_F32) LAUNCH(float);
   else if (dtype == NHV_BF16) LAUNCH(__nv_bfloat16);
   else NHV_REQUIRE(false, "latent_rope_store: unknown dtype %d", dtype);

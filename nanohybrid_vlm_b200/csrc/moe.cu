@@ -6,13 +6,15 @@
 //                 neighbours, a group's score is its largest c, and only outputs of the `keep` best groups can be
 //                 chosen (the others count as -inf); the `top` outputs with the largest c are chosen; their weights
 //                 are their s, divided by the sum of the chosen s (+ 1e-20).  One warp per token, all in fp32.
-//                 sigmoid_scores: s = sigmoid(z) instead of the softmax; renorm 0: the weights are the chosen s as
-//                 they are.
+//                 scores 1: s = sigmoid(z) instead of the softmax; renorm 0: the weights are the chosen s as they are.
+//                 scores 2: s = c = z + correction (a bias of the logits), and the weights are the softmax over the
+//                 chosen alone.
 //   moe_align     slots (t, k) whose choice is a real expert are grouped by expert; each expert's run is padded to
 //                 a multiple of the row tile, so that a tile of rows has one expert.  Writes sorted_slots (slot per
 //                 row, -1 for padding), slot_pos (row per slot, -1 for identity choices) and tile_expert.
 //   moe_gemm      (any type, CUDA cores, fixed order of summation over k) the products over the sorted rows:
-//                 first: act[row] = glu(x[token(row)] Wg[e]^T, x[token(row)] Wu[e]^T), second: y[row] = act[row] Wd[e]^T.
+//                 first: act[row] = glu(x[token(row)] Wg[e]^T, x[token(row)] Wu[e]^T), or relu(x[token(row)] Wu[e]^T)^2 for
+//                 experts without a gate; second: y[row] = act[row] Wd[e]^T.
 //                 row_scale [slots] (optional): a factor on the expert's input, one per (token, choice) slot; it is
 //                 applied to both first products' fp32 sums, which equals scaling the input.
 //   moe_combine   out[t] = sum_k w[t,k] * (choice is an expert ? y[row(t,k)] : x[t]) + sigmoid(sg[t]) * shared[t];
@@ -39,7 +41,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 
 __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits, int ld,
-    const float* __restrict__ correction, int n_tokens, int N, int n_groups, int keep, int top, int sigmoid_scores,
+    const float* __restrict__ correction, int n_tokens, int N, int n_groups, int keep, int top, int scores,
     int renorm) {
   extern __shared__ float smem[];
   pdl_prologue();
@@ -50,7 +52,9 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
   float* c = s + N;                          // choice scores
   float* gs = c + N;                         // group scores
   const float* z = logits + (size_t)t * ld;
-  if (sigmoid_scores) {
+  if (scores == 2) {
+    for (int j = lane; j < N; j += 32) s[j] = c[j] = z[j] + (correction ? correction[j] : 0.f);
+  } else if (scores == 1) {
     for (int j = lane; j < N; j += 32) {
       const float v = 1.0f / (1.0f + expf(-z[j]));
       s[j] = v;
@@ -97,7 +101,7 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
       if (gs[j / gsz] != INFINITY) c[j] = -INFINITY;
     __syncwarp();
   }
-  float wsum = 0.f;
+  float wsum = 0.f, best = 0.f;
   for (int r = 0; r < top; ++r) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -107,7 +111,11 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     }
     warp_argmax(bv, bi);
     if (bi >= N) bi = 0;                                       // nothing left to choose: a configuration fault
-    const float w = s[bi];
+    float w = s[bi];
+    if (scores == 2) {                                         // the first chosen is the largest: no exponent is positive
+      if (r == 0) best = w;
+      w = expf(w - best);
+    }
     wsum += w;
     if (lane == 0) {
       ids[(size_t)t * top + r] = bi;
@@ -116,15 +124,17 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     }
     __syncwarp();
   }
-  if (!renorm) return;
-  const float inv = 1.0f / (wsum + 1e-20f);
+  if (!renorm && scores != 2) return;
+  __syncwarp();
+  const float inv = 1.0f / (wsum + (scores == 2 ? 0.f : 1e-20f));
   for (int r = lane; r < top; r += 32) weights[(size_t)t * top + r] *= inv;
 }
 
 NHV_API int nhv_moe_route(int* ids, float* weights, const float* logits, int ld, const float* correction, int n_tokens, int N,
-                          int n_groups, int keep, int top, int sigmoid_scores, int renorm, cudaStream_t stream) {
+                          int n_groups, int keep, int top, int scores, int renorm, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   NHV_REQUIRE(N > 0 && N <= 4096 && top > 0 && top <= N && ld >= N, "moe_route: bad sizes (N %d, top %d)", N, top);
+  NHV_REQUIRE(scores >= 0 && scores <= 2, "moe_route: unknown kind of scores %d", scores);
   NHV_REQUIRE(n_groups > 0 && N % n_groups == 0 && keep > 0 && keep <= n_groups,
               "moe_route: %d outputs do not form %d equal groups of which %d are kept", N, n_groups, keep);
   NHV_REQUIRE((long)keep * (N / n_groups) >= top, "moe_route: the kept groups hold fewer than top = %d outputs", top);
@@ -132,7 +142,7 @@ NHV_API int nhv_moe_route(int* ids, float* weights, const float* logits, int ld,
   if (smem > 48 * 1024)
     NHV_CUDA(cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "moe_route");
   nhv_launch(moe_route_kernel, (n_tokens + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, smem, stream, ids, weights, logits, ld,
-             correction, n_tokens, N, n_groups, keep, top, sigmoid_scores, renorm);
+             correction, n_tokens, N, n_groups, keep, top, scores, renorm);
   NHV_CHECK_LAUNCH("moe_route");
   return 0;
 }
@@ -208,13 +218,14 @@ constexpr int MG_BK = 32;
 #include "nhv_glu.cuh"
 
 
-// FIRST: A rows are x[sorted_slots[row] / top], B = (Wg[e], Wu[e]) [N, K] each, out = glu.  Else: A rows are
-// a[row], B = Wd[e] [N, K].  256 threads: thread (ty, tx) has rows ty * 4 .. + 3 of column tx.
-template <typename T, bool FIRST>
+// MODE 1: A rows are x[sorted_slots[row] / top], B = (Wg[e], Wu[e]) [N, K] each, out = glu.  MODE 2: the same rows, B =
+// Wu[e], out = relu^2.  MODE 0: A rows are a[row], B = Wd[e] [N, K].  256 threads: thread (ty, tx) has rows ty * 4 .. + 3 of column tx.
+template <typename T, int MODE>
 __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(
     T* __restrict__ out, const T* __restrict__ A, int lda, const T* __restrict__ W0, const T* __restrict__ W1,
     const int* __restrict__ sorted_slots, const int* __restrict__ tile_expert, int top, int N, int K, float limit,
     float alpha, float up_shift, const float* __restrict__ row_scale) {
+  constexpr bool FIRST = MODE == 1, GATHER = MODE != 0;
   __shared__ float As[MG_BM][MG_BK + 1];
   __shared__ float ascale[MG_BM];
   __shared__ float B0[MG_BN][MG_BK + 1];
@@ -228,8 +239,8 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(
   if (tid < MG_BM) {
     const int row = tile * MG_BM + tid;
     const int slot = sorted_slots[row];
-    arow[tid] = slot < 0 ? -1 : (FIRST ? slot / top : row);
-    ascale[tid] = (FIRST && row_scale && slot >= 0) ? row_scale[slot] : 1.f;
+    arow[tid] = slot < 0 ? -1 : (GATHER ? slot / top : row);
+    ascale[tid] = (GATHER && row_scale && slot >= 0) ? row_scale[slot] : 1.f;
   }
   __syncthreads();
   const T* w0 = W0 + (size_t)e * N * K;
@@ -269,16 +280,17 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(
     const size_t row = (size_t)tile * MG_BM + lr;
     // the storage type's rounding of gate and up comes first, as a separate product would leave it
     const float sc = ascale[lr];          // a factor on the expert's input is a factor on both first products
-    const float v = FIRST ? nhv_glu(round_to<T>(sc * acc0[r]), round_to<T>(sc * acc1[r]), limit, alpha, up_shift) : acc0[r];
+    const float v = FIRST ? nhv_glu(round_to<T>(sc * acc0[r]), round_to<T>(sc * acc1[r]), limit, alpha, up_shift)
+                          : (MODE == 2 ? nhv_relu_squared_unit(round_to<T>(sc * acc0[r])) : acc0[r]);
     out[row * N + n0 + tx] = from_f32<T>(v);
   }
 }
 
 NHV_API int nhv_moe_simt_tile() { return MG_BM; }
 
-// first != 0: out [rows, N] = glu over x [T, K] gathered by sorted_slots, W0 / W1 [E, N, K].  first == 0: out [rows, N]
-// = a [rows, K] times W0 [E, N, K].  max_tiles: the tiles of the ordering (rows / tile).
-NHV_API int nhv_moe_gemm_simt(int dtype, int first, void* out, const void* A, int lda, const void* W0, const void* W1,
+// mode 1: out [rows, N] = glu over x [T, K] gathered by sorted_slots, W0 / W1 [E, N, K]; 2: relu^2 of the same rows times
+// W0 [E, N, K]; 0: out [rows, N] = a [rows, K] times W0 [E, N, K].  max_tiles: the tiles of the ordering (rows / tile).
+NHV_API int nhv_moe_gemm_simt(int dtype, int mode, void* out, const void* A, int lda, const void* W0, const void* W1,
                               const int* sorted_slots, const int* tile_expert, int max_tiles, int top, int N, int K,
                               float limit, float alpha, float up_shift, const float* row_scale, cudaStream_t stream) {
   if (max_tiles == 0) return 0;
@@ -288,8 +300,8 @@ NHV_API int nhv_moe_gemm_simt(int dtype, int first, void* out, const void* A, in
 #define GO(T, F)                                                                                                 \
   nhv_launch(moe_gemm_simt_kernel<T, F>, grid, 256, 0, stream, (T*)out, (const T*)A, lda, (const T*)W0, (const T*)W1, \
              sorted_slots, tile_expert, top, N, K, limit, alpha, up_shift, row_scale)
-  if (dtype == NHV_F32) { if (first) GO(float, true); else GO(float, false); }
-  else if (dtype == NHV_BF16) { if (first) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
+  if (dtype == NHV_F32) { if (mode == 1) GO(float, 1); else if (mode == 2) GO(float, 2); else GO(float, 0); }
+  else if (dtype == NHV_BF16) { if (mode == 1) GO(__nv_bfloat16, 1); else if (mode == 2) GO(__nv_bfloat16, 2); else GO(__nv_bfloat16, 0); }
   else NHV_REQUIRE(false, "moe_gemm: unknown dtype %d", dtype);
 #undef GO
   NHV_CHECK_LAUNCH("moe_gemm");

@@ -6,7 +6,8 @@
 //   first:  act[row, c] = glu(x[token(row)] . Wg[e][c], x[token(row)] . Wu[e][c])   64 columns: 64 gate rows and the 64
 //           up rows of the same columns lie in one 128-row tile of B, and a warp's fragments hold gate and up of the
 //           same (row, column) in the same thread, so the unit is applied without leaving the registers;
-//   second: y[row, c] = act[row] . Wd[e][c]                                          128 columns.
+//   second: y[row, c] = act[row] . Wd[e][c]                                          128 columns;
+//   for experts without a gate, first: act[row, c] = relu(x[token(row)] . Wu[e][c])^2   128 columns.
 // A rows are gathered by token on their way into shared memory.  Operands travel by cp.async in a ring of three
 // stages of 32 columns of K (small stages: several blocks fit an SM, and the tensor pipe needs many warps to stay
 // busy); a row's sum over K runs in the same order wherever the row stands, so results do not depend on the
@@ -50,11 +51,12 @@ template <int BM> struct MmShape {
   static constexpr int THREADS = (BM / WM) * 4 * 32;   // warps: BM / WM along the rows x 4 along the columns
 };
 
-template <int BM, bool FIRST>
+template <int BM, int MODE>
 __global__ void __launch_bounds__(MmShape<BM>::THREADS) moe_gemm_mma_kernel(
     bf16* __restrict__ out, const bf16* __restrict__ A, int lda, const bf16* __restrict__ W0, const bf16* __restrict__ W1,
     const int* __restrict__ sorted_slots, const int* __restrict__ tile_expert, int top, int N, int K, float limit,
     float alpha, float up_shift, const float* __restrict__ row_scale) {
+  constexpr bool FIRST = MODE == 1, GATHER = MODE != 0;
   constexpr int MT = MmShape<BM>::WM / 16, MM_THREADS = MmShape<BM>::THREADS;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* As = reinterpret_cast<bf16*>(smem_raw);              // [STAGES][BM][LDS]
@@ -72,8 +74,8 @@ __global__ void __launch_bounds__(MmShape<BM>::THREADS) moe_gemm_mma_kernel(
   if (tid < BM) {
     const int row = tile * BM + tid;
     const int slot = sorted_slots[row];
-    arow[tid] = slot < 0 ? -1 : (FIRST ? slot / top : row);
-    ascale[tid] = (FIRST && row_scale && slot >= 0) ? row_scale[slot] : 1.f;
+    arow[tid] = slot < 0 ? -1 : (GATHER ? slot / top : row);
+    ascale[tid] = (GATHER && row_scale && slot >= 0) ? row_scale[slot] : 1.f;
   }
   __syncthreads();
   const bf16* w0 = W0 + (size_t)e * N * K;
@@ -160,6 +162,9 @@ __global__ void __launch_bounds__(MmShape<BM>::THREADS) moe_gemm_mma_kernel(
           // gate and up rounded to the storage type first, as a separate product would leave them
           v0 = nhv_glu(mm_round(sc * acc[mt][j][2 * half]), mm_round(sc * acc[mt][j + 2][2 * half]), limit, alpha, up_shift);
           v1 = nhv_glu(mm_round(sc * acc[mt][j][2 * half + 1]), mm_round(sc * acc[mt][j + 2][2 * half + 1]), limit, alpha, up_shift);
+        } else if (MODE == 2) {
+          v0 = nhv_relu_squared_unit(mm_round(sc * acc[mt][j][2 * half]));
+          v1 = nhv_relu_squared_unit(mm_round(sc * acc[mt][j][2 * half + 1]));
         } else {
           v0 = acc[mt][j][2 * half];
           v1 = acc[mt][j][2 * half + 1];
@@ -174,20 +179,21 @@ __global__ void __launch_bounds__(MmShape<BM>::THREADS) moe_gemm_mma_kernel(
 template <int BM>
 static size_t mm_smem_bytes() { return (size_t)MM_STAGES * (BM + MM_BROWS) * MM_LDS * sizeof(bf16); }
 
-// tile: 16, 64 or 128, the row tile that moe_align was called with.  first != 0: out [rows, N] = glu over x [T, K] gathered
-// by sorted_slots, W0 / W1 [E, N, K]; first == 0: out [rows, N] = a [rows, K] times W0 [E, N, K].
-NHV_API int nhv_moe_gemm_mma(int tile, int first, void* out, const void* A, int lda, const void* W0, const void* W1,
+// tile: 16, 64 or 128, the row tile that moe_align was called with.  mode 1: out [rows, N] = glu over x [T, K] gathered
+// by sorted_slots, W0 / W1 [E, N, K]; 2: relu^2 of the same rows times W0; 0: out [rows, N] = a [rows, K] times W0 [E, N, K].
+NHV_API int nhv_moe_gemm_mma(int tile, int mode, void* out, const void* A, int lda, const void* W0, const void* W1,
                              const int* sorted_slots, const int* tile_expert, int max_tiles, int top, int N, int K,
                              float limit, float alpha, float up_shift, const float* row_scale, cudaStream_t stream) {
   if (max_tiles == 0) return 0;
   NHV_REQUIRE(tile == 16 || tile == 64 || tile == 128, "moe_gemm (mma): the row tile is 16, 64 or 128, not %d", tile);
   NHV_REQUIRE(max_tiles > 0 && N > 0 && K > 0 && top > 0, "moe_gemm (mma): bad sizes");
   NHV_REQUIRE(K % 8 == 0 && lda % 8 == 0 && N % 2 == 0 && ((uintptr_t)A % 16) == 0 && ((uintptr_t)W0 % 16) == 0 &&
-                  (!first || ((uintptr_t)W1 % 16) == 0) && ((uintptr_t)out % 4) == 0,
+                  (mode != 1 || ((uintptr_t)W1 % 16) == 0) && ((uintptr_t)out % 4) == 0,
               "moe_gemm (mma): rows of A and of the weights must start on 16-byte boundaries (K %d, lda %d)", K, lda);
-  dim3 grid((N + (first ? 64 : 128) - 1) / (first ? 64 : 128), max_tiles);
+  const int panel = mode == 1 ? 64 : 128;
+  dim3 grid((N + panel - 1) / panel, max_tiles);
   NHV_REQUIRE(grid.y <= 65535, "moe_gemm (mma): %d tiles of rows are beyond the grid's reach", max_tiles);
-#define GO(BM, F)                                                                                                     \
+#define GO(BM, F)                                                                                                    \
   do {                                                                                                                \
     static bool attr = false;                                                                                         \
     if (!attr) {                                                                                                      \
@@ -199,9 +205,11 @@ NHV_API int nhv_moe_gemm_mma(int tile, int first, void* out, const void* A, int 
                lda, (const bf16*)W0, (const bf16*)W1, sorted_slots, tile_expert, top, N, K, limit, alpha, up_shift,   \
                row_scale);                                                                                            \
   } while (0)
-  if (tile == 16) { if (first) GO(16, true); else GO(16, false); }
-  else if (tile == 64) { if (first) GO(64, true); else GO(64, false); }
-  else { if (first) GO(128, true); else GO(128, false); }
+#define PICK(BM) do { if (mode == 1) GO(BM, 1); else if (mode == 2) GO(BM, 2); else GO(BM, 0); } while (0)
+  if (tile == 16) PICK(16);
+  else if (tile == 64) PICK(64);
+  else PICK(128);
+#undef PICK
 #undef GO
   NHV_CHECK_LAUNCH("moe_gemm (mma)");
   return 0;

@@ -7,7 +7,8 @@
 //   first:  the panel is 64 rows of the gate matrix and the 64 rows of the up matrix of the same output columns;
 //           act[row, c] = glu(gate, up): the lanes that hold up hand their numbers to the lanes that hold gate through
 //           shared memory (the ring, which is free by then);
-//   second: y[row, c] = act[row] . Wd[e][c], 128 output columns.
+//   second: y[row, c] = act[row] . Wd[e][c], 128 output columns;
+//   for experts without a gate, first: act[row, c] = relu(x[token(row)] . Wu[e][c])^2, 128 output columns.
 // The first product reads its A rows from a copy of x gathered into the order of the rows (moe_gather_rows below), so
 // that a tile of rows is one TMA box.
 //
@@ -104,8 +105,9 @@ struct alignas(64) Params {
   const float* row_scale;     // a factor on the expert's input per (token, choice) slot, or null
 };
 
-template <bool FIRST>
+template <int MODE>
 __global__ void __launch_bounds__(THREADS, 1) moe_tcgen05_kernel(const __grid_constant__ Params p) {
+  constexpr bool FIRST = MODE == 1;
   extern __shared__ unsigned char smem_unaligned[];
   unsigned char* smem = smem_unaligned + ((1024 - (smem_u32(smem_unaligned) & 1023)) & 1023);
   unsigned char* ring = smem;
@@ -194,7 +196,7 @@ __global__ void __launch_bounds__(THREADS, 1) moe_tcgen05_kernel(const __grid_co
       {
         const int slot = p.sorted_slots[(size_t)tile * ROWS + tid];
         s_live[tid] = slot >= 0;
-        s_scale[tid] = (FIRST && p.row_scale && slot >= 0) ? p.row_scale[slot] : 1.f;
+        s_scale[tid] = (MODE != 0 && p.row_scale && slot >= 0) ? p.row_scale[slot] : 1.f;
       }
       if (!mbar_wait(acc_full, 0, 4)) s_epi_abort = 1;
       epi_sync();
@@ -231,7 +233,9 @@ __global__ void __launch_bounds__(THREADS, 1) moe_tcgen05_kernel(const __grid_co
             if (n < p.N) {
 #pragma unroll
               for (int j = 0; j < 32; ++j)
-                if (s_live[c0 + j]) p.out[((size_t)tile * ROWS + c0 + j) * p.N + n] = __float2bfloat16_rn(v[j]);
+                if (s_live[c0 + j])
+                  p.out[((size_t)tile * ROWS + c0 + j) * p.N + n] =
+                      __float2bfloat16_rn(MODE == 2 ? nhv_relu_squared_unit(round_bf16(s_scale[c0 + j] * v[j])) : v[j]);
             }
           }
         }
@@ -306,20 +310,20 @@ NHV_API int nhv_moe_gather_rows(void* out, const void* x, const int* sorted_slot
   return 0;
 }
 
-// first != 0: out [rows, N] = glu(A W0[e]^T, A W1[e]^T) with A [rows, K] (the gathered rows) and W0 / W1 [E, N, K];
-// first == 0: out [rows, N] = A W0[e]^T.  rows = tiles * 128, the ordering of moe_align with tiles of 128 rows.
-NHV_API int nhv_moe_gemm_tcgen05(int first, void* out, const void* A, const void* W0, const void* W1, int n_experts,
+// mode 1: out [rows, N] = glu(A W0[e]^T, A W1[e]^T) with A [rows, K] (the gathered rows) and W0 / W1 [E, N, K]; 2: out =
+// relu(A W0[e]^T)^2 of the same rows; 0: out [rows, N] = A W0[e]^T.  rows = tiles * 128, the ordering of moe_align with tiles of 128 rows.
+NHV_API int nhv_moe_gemm_tcgen05(int mode, void* out, const void* A, const void* W0, const void* W1, int n_experts,
                                  const int* sorted_slots, const int* tile_expert, int tiles, int N, int K, float limit,
                                  float alpha, float up_shift, const float* row_scale, cudaStream_t stream) {
   if (tiles == 0) return 0;
   NHV_REQUIRE(tiles > 0 && N > 0 && K > 0 && K % 8 == 0 && n_experts > 0, "moe_gemm (tcgen05): K must be a multiple of 8 (N=%d K=%d)", N, K);
-  NHV_REQUIRE(((uintptr_t)A % 16) == 0 && ((uintptr_t)W0 % 16) == 0 && (!first || ((uintptr_t)W1 % 16) == 0),
+  NHV_REQUIRE(((uintptr_t)A % 16) == 0 && ((uintptr_t)W0 % 16) == 0 && (mode != 1 || ((uintptr_t)W1 % 16) == 0),
               "moe_gemm (tcgen05): operands must be 16-byte aligned");
   NHV_REQUIRE((long long)n_experts * N < (1LL << 31) && (long long)tiles * ROWS < (1LL << 31), "moe_gemm (tcgen05): too many rows");
   Params p;
-  const int box = first ? PANEL / 2 : PANEL;
+  const int box = mode == 1 ? PANEL / 2 : PANEL;
   NHV_REQUIRE(weight_map(&p.w0_map, W0, (long long)n_experts * N, K, box), "moe_gemm (tcgen05): cannot encode the weights' tensor map");
-  if (first) NHV_REQUIRE(weight_map(&p.w1_map, W1, (long long)n_experts * N, K, box), "moe_gemm (tcgen05): cannot encode the weights' tensor map");
+  if (mode == 1) NHV_REQUIRE(weight_map(&p.w1_map, W1, (long long)n_experts * N, K, box), "moe_gemm (tcgen05): cannot encode the weights' tensor map");
   else p.w1_map = p.w0_map;
   NHV_REQUIRE(nhv_make_map_bf16(&p.a_map, A, (long long)tiles * ROWS, K, K, BK, ROWS), "moe_gemm (tcgen05): cannot encode the rows' tensor map");
   p.out = (bf16*)out;
@@ -335,11 +339,13 @@ NHV_API int nhv_moe_gemm_tcgen05(int first, void* out, const void* A, const void
   NHV_REQUIRE(grid.y <= 65535, "moe_gemm (tcgen05): %d tiles of rows are beyond the grid's reach", tiles);
   static bool attr_set = false;
   if (!attr_set) {
-    NHV_CUDA(cudaFuncSetAttribute(moe_tcgen05_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES), "moe_gemm (tcgen05)");
-    NHV_CUDA(cudaFuncSetAttribute(moe_tcgen05_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES), "moe_gemm (tcgen05)");
+    NHV_CUDA(cudaFuncSetAttribute(moe_tcgen05_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES), "moe_gemm (tcgen05)");
+    NHV_CUDA(cudaFuncSetAttribute(moe_tcgen05_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES), "moe_gemm (tcgen05)");
+    NHV_CUDA(cudaFuncSetAttribute(moe_tcgen05_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES), "moe_gemm (tcgen05)");
     attr_set = true;
   }
-  if (first) NHV_CUDA(nhv_launch(moe_tcgen05_kernel<true>, grid, dim3(THREADS), SMEM_BYTES, stream, p), "moe_gemm (tcgen05)");
-  else NHV_CUDA(nhv_launch(moe_tcgen05_kernel<false>, grid, dim3(THREADS), SMEM_BYTES, stream, p), "moe_gemm (tcgen05)");
+  if (mode == 1) NHV_CUDA(nhv_launch(moe_tcgen05_kernel<1>, grid, dim3(THREADS), SMEM_BYTES, stream, p), "moe_gemm (tcgen05)");
+  else if (mode == 2) NHV_CUDA(nhv_launch(moe_tcgen05_kernel<2>, grid, dim3(THREADS), SMEM_BYTES, stream, p), "moe_gemm (tcgen05)");
+  else NHV_CUDA(nhv_launch(moe_tcgen05_kernel<0>, grid, dim3(THREADS), SMEM_BYTES, stream, p), "moe_gemm (tcgen05)");
   return 0;
 }

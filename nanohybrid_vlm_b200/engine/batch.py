@@ -62,6 +62,9 @@ class StepBatch:
     temperatures: torch.Tensor | None = None    # [R] float32
     seeds: torch.Tensor | None = None           # [R] int64
     sample_positions: torch.Tensor | None = None  # [R] int32: the position of the token being chosen
+    # what one layer of this step leaves for later ones (values that later layers mix in, plans that layers share),
+    # under a key that the parts agree on; it ends with the step
+    carried: dict = field(default_factory=dict)
 
 
 def _align(n: int, a: int = 4) -> int:

@@ -59,15 +59,15 @@ _SIGNATURES = {
     "nhv_moe_combine": [I, P, P, P, P, P, I, P, P, P, I, I, I, I, P],
     "nhv_attention_simt_ex": [I, P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, I, I, P],
     "nhv_causal_filter_add": [I, P, P, I, P, I, P, P, P, ctypes.c_long, P, P, P, I, I, I, I, P],
-    "nhv_latent_rope_store": [I, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P],
+    "nhv_latent_rope_store": [I, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, I, P],
     "nhv_gemm_nt_simt_batched": [I, P, P, P, I, I, I, I, I, I, I, I, ctypes.c_long, ctypes.c_long, ctypes.c_long, P],
     "nhv_general_delta": [I, P, P, I, P, I, P, P, P, P, ctypes.c_long, P, P, P, P, P, P, I, I, I, I, F, P],
     "nhv_general_delta_tanh": [I, P, P, I, I, I, P],
     "nhv_sigmoid_mul_heads": [I, P, I, P, I, P, I, I, I, I, I, P],
-    "nhv_latent_gather": [I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, P],
+    "nhv_latent_gather": [I, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, P],
     "nhv_latent_assemble": [I, P, P, P, P, P, I, P, I, ctypes.c_long, I, I, I, I, I, I, I, P],
     "nhv_latent_decode_supports": [I, I, I],
-    "nhv_latent_decode": [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, F, P, I, P, P, P],
+    "nhv_latent_decode": [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, F, I, P, I, P, P, P],
     "nhv_relu_squared": [I, P, c_size_t, P],
     "nhv_scale_softcap": [P, F, F, c_size_t, P],
     "nhv_gelu_tanh": [I, P, c_size_t, P],
@@ -75,6 +75,8 @@ _SIGNATURES = {
     "nhv_stream_round": [I, P, P, c_size_t, P],
     "nhv_token_shift_mix": [I, P, P, P, P, ctypes.c_long, P, P, P, I, I, I, I, P],
     "nhv_decay_scan": [I, P, P, P, P, I, P, P, P, P, ctypes.c_long, P, P, P, I, I, I, I, I, I, I, P],
+    "nhv_streams_rmsnorm": [I, P, P, P, I, P, P, P, P, P, P, I, I, I, F, P],
+    "nhv_row_norm_store": [I, P, I, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, P, P],
     "nhv_decay_lowrank": [I, P, P, I, P, P, I, I, I, P],
 }
 

@@ -135,6 +135,28 @@ def rmsnorm_stream(out, stream, weight, eps: float, addends=(), rows=None, write
          float(weight_offset), int(groups), stream_ptr())
 
 
+def streams_rmsnorm(out, dst, src, weight, eps: float, y=None, mix=None, write=None, read=None, rows=None,
+                    n_streams: int | None = None) -> None:
+    """The norm over a residual stream kept as S float32 copies per token.  src [T, S, width], or [T, 1, width] while all
+    copies are equal (``n_streams`` then says S).  With a sub-block's output ``y`` [T, width] the copies are rebuilt
+    first: x'_t = sum_s mix[s, t] x_s + write[t] y, stored to ``dst`` [T, S, width] (None: not kept; ``src`` itself: in
+    place).  out[r] = u / rms(u) * weight of u = sum_t read[t] x'_t (``read`` None: the plain sum), src row rows[r] or r.
+    mix [S, S] indexed [from, to], write and read [S]: float32.  All sums in 32-bit, one rounding."""
+    _need_cuda(out, dst, src, weight, y, mix, write, read, rows)
+    _contig("out", out); _contig("streams", src)
+    T, given, width = src.shape
+    S = n_streams or given
+    assert given in (1, S) and src.dtype == torch.float32 and weight.numel() == width and weight.dtype == out.dtype
+    for t, n in ((mix, S * S), (write, S), (read, S)):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == n and t.is_contiguous())
+    assert y is None or (y.shape == (T, width) and y.dtype == out.dtype and y.is_contiguous() and mix is not None)
+    assert dst is None or (dst.shape == (T, S, width) and dst.dtype == torch.float32 and dst.is_contiguous())
+    n_rows = rows.numel() if rows is not None else T
+    assert out.numel() == n_rows * width and (rows is None or rows.dtype == torch.int32)
+    call("nhv_streams_rmsnorm", dtype_code(out), out.data_ptr(), _ptr(dst), src.data_ptr(), given, _ptr(y), _ptr(mix),
+         _ptr(write), _ptr(read), weight.data_ptr(), _ptr(rows), n_rows, S, width, float(eps), stream_ptr())
+
+
 def scaled_sum(out, a, b, ca: float, cb: float) -> None:
     """out = ca * a + cb * b elementwise (sums in 32-bit)."""
     _need_cuda(out, a, b)
@@ -278,11 +300,12 @@ def causal_filter_add(out1, out2, x, w1, w2, state, batch) -> None:
 
 
 def latent_rope_store(kv, q, q_lat, pages, slot_mapping, positions, cos_sin, rotary_dim: int, H: int, dn: int, dr: int,
-                      rank: int, eps: float, weight) -> None:
+                      rank: int, eps: float, weight, interleaved: bool = False) -> None:
     """For attention over one latent vector per token.  kv [T, rank + dr] (a view with unit column stride): the first
     ``rank`` elements normed (unit root mean square, times ``weight`` [rank]) and the last dr rotated go to the token's
     row of ``pages`` [pages, 1, 1, page_size, row >= rank + dr] (None: nothing is stored).  q [T, H * (dn + dr)]: every
-    head's last dr elements, rotated, go to q_lat [T, H * (rank + dr)] behind the head's first ``rank`` places."""
+    head's last dr elements, rotated, go to q_lat [T, H * (rank + dr)] behind the head's first ``rank`` places.
+    ``interleaved``: element 2i turns with element 2i + 1 instead of element i with element i + rotary_dim / 2."""
     _need_cuda(kv, q, q_lat, pages, slot_mapping, positions, cos_sin, weight)
     T = kv.shape[0]
     assert kv.stride(1) == 1 and kv.shape[1] == rank + dr and q.stride(1) == 1 and q.shape == (T, H * (dn + dr))
@@ -301,7 +324,7 @@ def latent_rope_store(kv, q, q_lat, pages, slot_mapping, positions, cos_sin, rot
     call("nhv_latent_rope_store", dtype_code(kv), kv.data_ptr(), kv.stride(0), q.data_ptr(), q.stride(0), q_lat.data_ptr(),
          q_lat.stride(0), _ptr(pages), _ptr(slot_mapping), _ptr(positions), _ptr(cos_sin), int(rotary_dim),
          0 if cos_sin is None else cos_sin.shape[0], T, H, dn, dr, rank, row, page_size, n_pages, float(eps),
-         weight.data_ptr(), stream_ptr())
+         weight.data_ptr(), int(bool(interleaved)), stream_ptr())
 
 
 def linear_heads(out, x, weight) -> None:
@@ -367,29 +390,50 @@ def sigmoid_mul_heads(out, x, gate, group: int, x_head: int | None = None) -> No
 LATENT_TILE = 64        # rows of a temporary page of expanded keys and values
 
 
-def latent_expand(pages, tables, batch, q, q_lat, ukv, H: int, dn: int, dr: int, dv: int, rank: int, D: int):
+def latent_tiles(host_cu_q, host_kv_len, window: int) -> list[tuple[int, int]]:
+    """Per request of a step: the tiles of 64 tokens [from, to) whose latents its new tokens see (all up to its last
+    token; with a window none before the tile of the first key that the first new token sees)."""
+    out = []
+    for s, n in enumerate(host_kv_len):
+        new = host_cu_q[s + 1] - host_cu_q[s]
+        lo = max(0, n - new - window + 1) if window > 0 else 0
+        out.append((lo // LATENT_TILE, -(-n // LATENT_TILE)))
+    return out
+
+
+def _latent_rows(batch, window: int, device):
+    """Where a step's latents go when they are expanded: per request the first temporary row and the first token, the
+    block tables of the temporary pages, how many pages, and the most rows of a request."""
+    tiles = latent_tiles(batch.host_cu_q, batch.host_kv_len, window)
+    width, at, rows0, table = max(b for _, b in tiles), 0, [], []
+    for a, b in tiles:
+        rows0.append(at * LATENT_TILE)
+        table.append([at + i - a if a <= i < b else -1 for i in range(width)])
+        at += b - a
+    flat = torch.tensor(rows0 + [a * LATENT_TILE for a, _ in tiles] + [p for row in table for p in row], dtype=torch.int32)
+    flat = (flat.pin_memory() if device.type == "cuda" else flat).to(device, non_blocking=True)
+    S = len(tiles)
+    return flat[:S], flat[S:2 * S], flat[2 * S:].view(S, width), at, max(b - a for a, b in tiles) * LATENT_TILE
+
+
+def latent_expand(pages, tables, batch, q, q_lat, ukv, H: int, dn: int, dr: int, dv: int, rank: int, D: int,
+                  window: int = 0):
     """Attention over one latent per token, prepared for the tensor-core kernels: the latents of the step's requests
-    (all their tokens in the cache) are expanded by ``ukv`` [H dn + H dv, rank] into a key [dn | rotated part dr | 0]
+    (all their tokens in the cache, or with a ``window`` those from the tile of the first key that one of the step's
+    tokens sees) are expanded by ``ukv`` [H dn + H dv, rank] into a key [dn | rotated part dr | 0]
     and a value [dv | 0] per head, padded to D elements, in temporary pages of 64 tokens; the queries likewise.
     Returns (queries [T, H D], temporary pages [n, 2, H, 64, D], their block tables [requests, pages])."""
     _need_cuda(pages, q, q_lat, ukv)
     T, row = q.shape[0], pages.shape[-1]
-    plan = getattr(batch, "_latent_rows", None)
-    if plan is None or plan[3] != batch.host_kv_len:        # every such layer of the step uses the same rows
-        counts = [-(-n // LATENT_TILE) for n in batch.host_kv_len]
-        first, width = [0], max(counts)
-        for c in counts:
-            first.append(first[-1] + c)
-        table = [[first[s] + i if i < counts[s] else -1 for i in range(width)] for s in range(len(counts))]
-        plan = (torch.tensor([f * LATENT_TILE for f in first[:-1]], dtype=torch.int32).to(q.device, non_blocking=True),
-                torch.tensor(table, dtype=torch.int32).to(q.device, non_blocking=True), first[-1], list(batch.host_kv_len))
-        batch._latent_rows = plan
-    row0, tmp_table, n_tmp = plan[:3]
+    plan = batch.carried.get(("latent_rows", window))
+    if plan is None:                                        # every such layer of the step uses the same rows
+        plan = batch.carried[("latent_rows", window)] = _latent_rows(batch, window, q.device)
+    row0, first, tmp_table, n_tmp, most = plan
     rows = n_tmp * LATENT_TILE
     lat = torch.empty(rows, rank, dtype=q.dtype, device=q.device)
     kr = torch.empty(rows, max(dr, 1), dtype=q.dtype, device=q.device)
     call("nhv_latent_gather", dtype_code(q), lat.data_ptr(), kr.data_ptr(), pages.data_ptr(), tables.block_tables.data_ptr(),
-         tables.block_tables.stride(0), batch.kv_len.data_ptr(), row0.data_ptr(), batch.n_seqs, batch.max_kv_len, rank, dr,
+         tables.block_tables.stride(0), batch.kv_len.data_ptr(), row0.data_ptr(), first.data_ptr(), batch.n_seqs, most, rank, dr,
          row, pages.shape[3], pages.shape[0], stream_ptr())
     kv = torch.empty(rows, ukv.shape[0], dtype=q.dtype, device=q.device)
     linear(kv, lat, ukv)
@@ -403,10 +447,12 @@ def latent_expand(pages, tables, batch, q, q_lat, ukv, H: int, dn: int, dr: int,
 LATENTS_ON_TENSOR_CORES = True      # tests switch it off to compare with the CUDA-core kernel at the same shapes
 
 
-def latent_attention(out, q_lat, pages, tables, batch, H: int, rank: int, row: int, scale: float, sinks=None) -> None:
+def latent_attention(out, q_lat, pages, tables, batch, H: int, rank: int, row: int, scale: float, sinks=None,
+                     window: int = 0) -> None:
     """Attention of the step's tokens over one latent per token: pages with one plane whose rows [row] are the key of
     every head and whose leading ``rank`` elements are the value of every head; q_lat [T, H row] -> out [T, H rank].
-    ``sinks`` [H] float32: exp(sink) joins each head's softmax denominator once.  bfloat16 with rows and latents in
+    ``sinks`` [H] float32: exp(sink) joins each head's softmax denominator once.  ``window`` > 0: the last ``window``
+    tokens only.  bfloat16 with rows and latents in
     steps of 8 runs on the tensor cores, a token's keys shared between blocks and merged (scratch: one partial result
     per token, head and piece); float32 and other sizes run the CUDA-core kernel."""
     _need_cuda(out, q_lat, pages, sinks)
@@ -414,17 +460,19 @@ def latent_attention(out, q_lat, pages, tables, batch, H: int, rank: int, row: i
     if not (LATENTS_ON_TENSOR_CORES and q_lat.dtype == torch.bfloat16 and pages.shape[1] == 1 and pages.shape[2] == 1
             and pages.shape[-1] == row and library.load_library().nhv_latent_decode_supports(H, rank, row)):
         attention_sink_simt(out, q_lat, pages, tables.block_tables, batch.cu_q, batch.kv_len, batch.n_seqs, batch.n_tokens,
-                            H, 1, row, rank, scale, sinks)
+                            H, 1, row, rank, scale, sinks, window)
         return
     _contig("kv_pages", pages)
     assert q_lat.shape == (T, H * row) and out.shape == (T, H * rank) and out.dtype == pages.dtype == torch.bfloat16
     assert q_lat.stride(1) == 1 and out.stride(1) == 1 and sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == H)
     tiles = -(-batch.max_kv_len // 64)
+    if window > 0:
+        tiles = min(tiles, (window + 62) // 64 + 1)          # a window lies over so many tiles at most
     pieces = max(1, min(tiles, 64, 2 * 148 // (T * -(-H // 16))))      # two rounds of blocks over the 148 SMs at most
     part = torch.empty(T * H * pieces * (rank + 2), dtype=torch.float32, device=out.device)
     call("nhv_latent_decode", out.data_ptr(), out.stride(0), q_lat.data_ptr(), q_lat.stride(0), pages.data_ptr(),
          tables.block_tables.data_ptr(), tables.block_tables.stride(0), batch.cu_q.data_ptr(), batch.kv_len.data_ptr(),
-         batch.n_seqs, T, H, rank, row, pages.shape[3], pages.shape[0], float(scale), _ptr(sinks), pieces,
+         batch.n_seqs, T, H, rank, row, pages.shape[3], pages.shape[0], float(scale), int(window), _ptr(sinks), pieces,
          part.data_ptr(), part.data_ptr() + 4 * T * H * pieces * rank, stream_ptr())
 
 
@@ -597,15 +645,17 @@ def moe_route(ids, weights, logits, correction, n_outputs: int, n_groups: int, k
     Scores are the softmax over all outputs; the choice is by score + correction among the outputs of the ``keep`` best
     of ``n_groups`` groups of neighbours (a group's score: its largest choice score); the weights are the chosen scores
     divided by their sum (+ 1e-20).  ``scores`` "sigmoid": each output's score is the sigmoid of its logit;
-    ``renorm`` False: the weights are the chosen scores as they are."""
-    assert scores in ("softmax", "sigmoid")
+    ``renorm`` False: the weights are the chosen scores as they are.  ``scores`` "chosen_softmax": the choice is by the
+    logit + correction (a bias), and the weights are the softmax of these over the chosen alone."""
+    kinds = ("softmax", "sigmoid", "chosen_softmax")
+    assert scores in kinds
     _need_cuda(ids, weights, logits, correction)
     T, top = ids.shape
     assert ids.dtype == torch.int32 and weights.dtype == logits.dtype == torch.float32 and weights.shape == ids.shape
     assert ids.is_contiguous() and weights.is_contiguous() and logits.stride(1) == 1 and logits.shape[0] == T
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == n_outputs)
     call("nhv_moe_route", ids.data_ptr(), weights.data_ptr(), logits.data_ptr(), logits.stride(0), _ptr(correction), T,
-         n_outputs, n_groups, keep, top, int(scores == "sigmoid"), int(bool(renorm)), stream_ptr())
+         n_outputs, n_groups, keep, top, kinds.index(scores), int(bool(renorm)), stream_ptr())
 
 
 MOE_TILE_SIMT = 16      # rows of one expert that a block of the CUDA-core products takes (MG_BM of csrc/moe.cu)
@@ -635,21 +685,28 @@ def moe_experts_simt(act, y, x, gate, up, down, sorted_slots, tile_expert, top: 
                      up_shift: float = 1.0, row_scale=None) -> None:
     """The experts' two products over the ordered rows on the CUDA cores, for any storage type and size, in a fixed order
     of summation: act [rows, ff] = glu(x[token] gate[e]^T, x[token] up[e]^T), y [rows, width] = act down[e]^T, with
-    gate / up [E, ff, width] and down [E, width, ff]."""
+    gate / up [E, ff, width] and down [E, width, ff].  ``gate`` None: act = relu(x[token] up[e]^T)^2."""
     _need_cuda(act, y, x, gate, up, down, sorted_slots, tile_expert)
     for name, t in (("act", act), ("y", y), ("x", x), ("gate", gate), ("up", up), ("down", down)):
-        _contig(name, t)
-    E, ff, width = gate.shape
-    assert up.shape == gate.shape and down.shape == (E, width, ff) and x.shape[1] == width
+        if t is not None:
+            _contig(name, t)
+    E, ff, width = up.shape
+    assert (gate is None or gate.shape == up.shape) and down.shape == (E, width, ff) and x.shape[1] == width
     assert act.shape == (sorted_slots.numel(), ff) and y.shape == (sorted_slots.numel(), width)
-    assert act.dtype == y.dtype == x.dtype == gate.dtype == up.dtype == down.dtype
+    assert act.dtype == y.dtype == x.dtype == up.dtype == down.dtype and (gate is None or gate.dtype == up.dtype)
+    mode, w0, w1 = _first_product(gate, up)
     tiles = tile_expert.numel()
     assert tiles * MOE_TILE_SIMT == sorted_slots.numel()
-    call("nhv_moe_gemm_simt", dtype_code(x), 1, act.data_ptr(), x.data_ptr(), width, gate.data_ptr(), up.data_ptr(),
+    call("nhv_moe_gemm_simt", dtype_code(x), mode, act.data_ptr(), x.data_ptr(), width, w0, w1,
          sorted_slots.data_ptr(), tile_expert.data_ptr(), tiles, top, ff, width, float(limit), float(alpha), float(up_shift),
          _ptr(row_scale), stream_ptr())
     call("nhv_moe_gemm_simt", dtype_code(x), 0, y.data_ptr(), act.data_ptr(), ff, down.data_ptr(), None,
          sorted_slots.data_ptr(), tile_expert.data_ptr(), tiles, top, width, ff, 0.0, 0.0, 0.0, None, stream_ptr())
+
+
+def _first_product(gate, up):
+    """(form of the experts' first product, its first and second matrix): 1 a gated unit, 2 the square of relu."""
+    return (2, up.data_ptr(), None) if gate is None else (1, gate.data_ptr(), up.data_ptr())
 
 
 MOE_ON_TENSOR_CORES = True      # tests switch it off to compare with the CUDA-core products at the same shapes
@@ -664,10 +721,10 @@ def moe_experts(x, gate, up, down, ids, limit: float, alpha: float, up_shift: fl
     where an expert sees about a hundred rows or more; mma.sync with tiles of 64 rows below that and of 16 where it
     sees few and the products stream the weights), everything else on the CUDA cores.
     The experts' unit is g' sigmoid(alpha g') (u' + up_shift) with g' = min(g, limit), u' = clamp(u, -limit, limit)
-    (limit inf, alpha 1, up_shift 0: silu(g) u).  ``row_scale`` [T, top] float32: a factor on each chosen expert's input.
+    (limit inf, alpha 1, up_shift 0: silu(g) u); with ``gate`` None it is relu(u)^2.  ``row_scale`` [T, top] float32: a factor on each chosen expert's input.
     Returns (y [rows, width], one row per slot that chose a real expert, and slot_pos [T * top] int32, the row of each
     slot or -1)."""
-    E, ff, width = gate.shape
+    E, ff, width = up.shape
     assert row_scale is None or (row_scale.dtype == torch.float32 and row_scale.is_contiguous() and row_scale.numel() == ids.numel())
     top = ids.shape[1]
     mma = MOE_ON_TENSOR_CORES and x.dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
@@ -684,12 +741,10 @@ def moe_experts(x, gate, up, down, ids, limit: float, alpha: float, up_shift: fl
         moe_experts_simt(act, y, x, gate, up, down, sorted_slots, tile_expert, top, limit, alpha, up_shift, row_scale)
         return y, slot_pos
     _need_cuda(x, gate, up, down, ids)
-    for name, t in (("x", x), ("gate", gate), ("up", up), ("down", down)):
-        _contig(name, t)
-    assert up.shape == gate.shape and down.shape == (E, width, ff) and x.shape[1] == width
-    assert gate.dtype == up.dtype == down.dtype == torch.bfloat16
+    _check_experts(x, gate, up, down)
+    mode, w0, w1 = _first_product(gate, up)
     tiles = tile_expert.numel()
-    call("nhv_moe_gemm_mma", tile, 1, act.data_ptr(), x.data_ptr(), width, gate.data_ptr(), up.data_ptr(),
+    call("nhv_moe_gemm_mma", tile, mode, act.data_ptr(), x.data_ptr(), width, w0, w1,
          sorted_slots.data_ptr(), tile_expert.data_ptr(), tiles, top, ff, width, float(limit), float(alpha), float(up_shift),
          _ptr(row_scale), stream_ptr())
     call("nhv_moe_gemm_mma", tile, 0, y.data_ptr(), act.data_ptr(), ff, down.data_ptr(), None,
@@ -697,23 +752,30 @@ def moe_experts(x, gate, up, down, ids, limit: float, alpha: float, up_shift: fl
     return y, slot_pos
 
 
+def _check_experts(x, gate, up, down) -> None:
+    E, ff, width = up.shape
+    for name, t in (("x", x), ("gate", gate), ("up", up), ("down", down)):
+        if t is not None:
+            _contig(name, t)
+            assert t.dtype == torch.bfloat16
+    assert (gate is None or gate.shape == up.shape) and down.shape == (E, width, ff) and x.shape[1] == width
+
+
 def _moe_experts_tcgen05(x, gate, up, down, ids, limit: float, alpha: float, up_shift: float = 1.0, row_scale=None):
     """``moe_experts`` for prompts in bfloat16: tiles of 128 rows per expert, the tokens' rows gathered into that order
     (so that a tile is one TMA box), both products with tcgen05.mma and tensor-memory accumulators."""
     _need_cuda(x, gate, up, down, ids)
-    for name, t in (("x", x), ("gate", gate), ("up", up), ("down", down)):
-        _contig(name, t)
-    E, ff, width = gate.shape
+    _check_experts(x, gate, up, down)
+    E, ff, width = up.shape
     top = ids.shape[1]
-    assert up.shape == gate.shape and down.shape == (E, width, ff) and x.shape[1] == width
-    assert x.dtype == gate.dtype == up.dtype == down.dtype == torch.bfloat16
+    mode, w0, w1 = _first_product(gate, up)
     sorted_slots, slot_pos, tile_expert = moe_align(ids, E, MOE_TCGEN05_TILE)
     rows, tiles = sorted_slots.numel(), tile_expert.numel()
     xs = torch.empty(rows, width, dtype=x.dtype, device=x.device)
     act = torch.empty(rows, ff, dtype=x.dtype, device=x.device)
     y = torch.empty(rows, width, dtype=x.dtype, device=x.device)
     call("nhv_moe_gather_rows", xs.data_ptr(), x.data_ptr(), sorted_slots.data_ptr(), rows, top, width, stream_ptr())
-    call("nhv_moe_gemm_tcgen05", 1, act.data_ptr(), xs.data_ptr(), gate.data_ptr(), up.data_ptr(), E, sorted_slots.data_ptr(),
+    call("nhv_moe_gemm_tcgen05", mode, act.data_ptr(), xs.data_ptr(), w0, w1, E, sorted_slots.data_ptr(),
          tile_expert.data_ptr(), tiles, ff, width, float(limit), float(alpha), float(up_shift), _ptr(row_scale), stream_ptr())
     call("nhv_moe_gemm_tcgen05", 0, y.data_ptr(), act.data_ptr(), down.data_ptr(), None, E, sorted_slots.data_ptr(),
          tile_expert.data_ptr(), tiles, width, ff, 0.0, 0.0, 0.0, None, stream_ptr())
@@ -768,6 +830,40 @@ def rope_norm_store(qkv, q_out, kv_pages, slot_mapping, positions, cos_sin, rota
          0 if cos_sin is None else cos_sin.shape[0], n_tokens, nq, nkv, dk, dv, row, page_size, n_pages,
          -1.0 if eps is None else float(eps), _ptr(bias), int(bool(values_from_keys)), _ptr(q_weight), _ptr(k_weight),
          int(bool(norm_first)), int(bool(interleaved)), stream_ptr())
+
+
+def row_norm_store(qkv, q_out, q_head: int, kv_pages, slot_mapping, positions, cos_sin, rotary_dim: int, nq: int, nkv: int,
+                   dk: int, dv: int, eps: float | None, q_weight=None, k_weight=None, interleaved: bool = False,
+                   v_first=None, v_share=None) -> None:
+    """qkv [T, nq*dk + nkv*dk + nkv*dv] -> q_out [T, nq * q_head] (q_head >= dk, zeros behind a head's dk elements) and
+    K / V rows in kv_pages [pages, 2, nkv, page_size, row] at slot_mapping, for layers that norm the whole query and the
+    whole key projection at once: each divided by the root mean square over all its heads (eps None: no norm) times
+    ``q_weight`` [nq*dk] / ``k_weight`` [nkv*dk], then rotated per head.  ``v_first`` [T, nkv*dv] (a view with unit
+    column stride) and ``v_share`` [1] float32: the stored values are (1 - share) v + share v_first."""
+    _need_cuda(qkv, q_out, kv_pages, slot_mapping, positions, cos_sin, q_weight, k_weight, v_first, v_share)
+    T = qkv.shape[0]
+    assert qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= (nq + nkv) * dk + nkv * dv and q_head >= dk
+    assert q_out.shape == (T, nq * q_head) and q_out.stride(1) == 1 and q_out.dtype == qkv.dtype
+    for w, n in ((q_weight, nq * dk), (k_weight, nkv * dk)):
+        assert w is None or (w.dtype == qkv.dtype and w.is_contiguous() and w.numel() == n and eps is not None)
+    assert (v_first is None) == (v_share is None)
+    assert v_first is None or (v_first.shape == (T, nkv * dv) and v_first.stride(1) == 1 and v_first.dtype == qkv.dtype
+                               and v_share.dtype == torch.float32 and v_share.numel() == 1)
+    if kv_pages is not None:
+        _contig("kv_pages", kv_pages)
+        n_pages, two, h, page_size, row = kv_pages.shape
+        assert two == 2 and h == nkv and row >= max(dk, dv) and kv_pages.dtype == qkv.dtype
+        assert slot_mapping.dtype == torch.int32 and slot_mapping.numel() >= T
+    else:
+        n_pages, page_size, row = 0, 0, max(dk, dv)
+    if cos_sin is not None:
+        assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1] == rotary_dim
+        assert positions.dtype == torch.int32
+    call("nhv_row_norm_store", dtype_code(qkv), qkv.data_ptr(), qkv.stride(0), q_out.data_ptr(), q_out.stride(0), q_head,
+         _ptr(kv_pages), _ptr(slot_mapping), _ptr(positions), _ptr(cos_sin), int(rotary_dim),
+         0 if cos_sin is None else cos_sin.shape[0], int(bool(interleaved)), T, nq, nkv, dk, dv, row, page_size, n_pages,
+         -1.0 if eps is None else float(eps), _ptr(q_weight), _ptr(k_weight), _ptr(v_first),
+         0 if v_first is None else v_first.stride(0), _ptr(v_share), stream_ptr())
 
 
 def attention_sink_simt(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: int, n_tokens: int, nq: int, nkv: int,

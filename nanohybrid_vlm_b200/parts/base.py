@@ -6,7 +6,7 @@ dtype, device); it declares its tensors (:class:`~.spec.ParamDecl`), receives th
 ``bind`` and then computes on device tensors.  No part knows which model it is in.
 
 Adding a part: subclass the interface, then ``MIXERS.register("name", Class)`` (or
-``FEED_FORWARDS``, ``NORMS``, ``POSITIONS``, ``FILTERS``, ``BLOCKS``, ``EMBEDDINGS``, ``HEADS``).  A model
+``FEED_FORWARDS``, ``NORMS``, ``POSITIONS``, ``FILTERS``, ``CONNECTIONS``, ``BLOCKS``, ``EMBEDDINGS``, ``HEADS``).  A model
 description refers to it as ``part("name", ...)``.
 """
 from __future__ import annotations
@@ -48,6 +48,7 @@ FEED_FORWARDS = Registry("feed-forward")
 NORMS = Registry("norm")
 POSITIONS = Registry("position encoding")
 FILTERS = Registry("input filter")
+CONNECTIONS = Registry("stream connection")
 BLOCKS = Registry("block arrangement")
 
 
@@ -177,10 +178,13 @@ class Pending:
     output as well as its input); the next norm applies it inside its own kernel where it can, else through
     :meth:`settled`.
     ``rounded``: the stream itself rounded to the model's type, where the block before has it at hand (nothing pending);
-    a block whose sub-blocks read the stream unnormed takes it from here instead of rounding the stream again."""
+    a block whose sub-blocks read the stream unnormed takes it from here instead of rounding the stream again.
+    ``connection``: the residual stream is several copies per token, [T, S, width], and the (single) term reaches them
+    through this :class:`StreamConnection`'s matrices; the next norm applies them."""
     terms: tuple = ()
     post: "Norm | None" = None
     rounded: "torch.Tensor | None" = None
+    connection: "StreamConnection | None" = None
 
     def settled(self) -> "Pending":
         """The same sum with ``post`` applied by that norm's own ``forward`` (rounded to the model's type)."""
@@ -227,6 +231,12 @@ class Norm(Part):
         """Norm of (x + residual) at the given rows only; nothing is written back."""
         raise NotImplementedError
 
+    def forward_streams(self, x: Pending, streams: torch.Tensor, connection: "StreamConnection"):
+        """For a residual stream of several copies, ``streams`` [T, S, width] float32 (or [T, 1, width] while they are
+        all equal): the pending output joins the copies through its own connection, and the sum that ``connection``
+        reads of the new copies is normed.  Returns (the normed sum, the new copies)."""
+        raise NotImplementedError
+
     def add_normed(self, terms: tuple, residual: torch.Tensor, side_eps=None, want_rounded: bool = True):
         """residual (float32, in place) += norm(sum of ``terms``), terms as ``Mixer.forward_normed_terms`` gives them: for
         blocks that norm a sub-block's output.  Returns the new stream rounded to the model's type (or None)."""
@@ -243,6 +253,16 @@ class InputFilter(Part):
 
     def forward(self, x: torch.Tensor, batch, state) -> torch.Tensor:
         raise NotImplementedError
+
+
+class StreamConnection(Part):
+    """How one sub-block is connected to a residual stream kept as ``streams`` copies: ``read`` [S] (the weights of the
+    sum that it reads), ``write`` [S] (how its output joins each copy) and ``mix`` [S, S] (indexed [from, to]: how the
+    copies are rebuilt from one another), float32 tensors."""
+    streams: int
+    read: torch.Tensor
+    write: torch.Tensor
+    mix: torch.Tensor
 
 
 class PositionEncoding(Part):

@@ -9,7 +9,9 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import BLOCKS, FEED_FORWARDS, FILTERS, MIXERS, NORMS, Block, CompositeNeed, Pending
+from .base import (BLOCKS, CONNECTIONS, FEED_FORWARDS, FILTERS, MIXERS, NORMS, Block, CompositeNeed, Pending,
+                   StreamConnection)
+from .spec import ParamDecl, Source
 
 
 class PreNormResidualBlock(Block):
@@ -141,6 +143,59 @@ class PostNormResidualBlock(Block):
         return Pending(rounded=x), residual
 
 
+class HyperConnection(StreamConnection):
+    """A sub-block's connection to S copies of the residual stream by learned constants.  Parameters: ``streams`` (S),
+    ``source`` (the checkpoint's prefix): the tensors ``<source>.in`` [S], ``<source>.out`` [S] and ``<source>.mix``
+    [S, S], kept in float32 (they enter the residual sum)."""
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.streams = int(spec["streams"])
+        self.source = spec["source"]
+        if self.streams < 1:
+            raise ValueError("a residual stream has at least one copy")
+
+    def params(self):
+        S, s = self.streams, self.source
+        return [ParamDecl(f"{s}.{name}", shape, init=init, storage="float32", sources=(Source(f"{s}.{name}", 0, S),))
+                for name, shape, init in (("in", (S,), "layer_scale"), ("out", (S,), "layer_scale"), ("mix", (S, S), "stream_mix"))]
+
+    def bind(self, tensors):
+        s = self.source
+        self.read, self.write, self.mix = (tensors[f"{s}.{name}"].contiguous() for name in ("in", "out", "mix"))
+
+
+class HyperConnectionBlock(Block):
+    """A residual stream of S copies x_1 .. x_S (float32, [T, S, width]) in the place of one: each sub-block reads
+    norm(sum_s in[s] x_s), and its output y makes new copies x_t <- sum_s mix[s, t] x_s + out[t] y, all from the old ones.
+    The sub-block's output is handed on as a :class:`Pending` with its connection; the next norm in line (this layer's
+    second, the next layer's first, or the model's last, which sums the copies) rebuilds the copies, sums and norms in
+    one kernel.  Until the first output joins all copies equal the embedding and are kept as one row.  A layer may have no
+    feed-forward (then also no second norm and connection)."""
+    SLOTS = {"mixer": MIXERS, "mixer_norm": NORMS, "mixer_connection": CONNECTIONS, "ffn": FEED_FORWARDS, "ffn_norm": NORMS,
+             "ffn_connection": CONNECTIONS}
+    OPTIONAL = ("ffn", "ffn_norm", "ffn_connection")
+
+    def __init__(self, spec, parts):
+        super().__init__(spec, parts)
+        has = [name in parts for name in self.OPTIONAL]
+        if any(has) and not all(has):
+            raise ValueError("a feed-forward comes with its norm and its connection, or not at all")
+
+    def forward(self, hidden, residual, batch, cache):
+        if residual is None:
+            residual = (hidden if hidden.dtype == torch.float32 else hidden.float()).unsqueeze(1)
+            hidden = Pending()
+        x, residual = self.mixer_norm.forward_streams(hidden, residual, self.mixer_connection)
+        pending = Pending(((self.mixer.forward(x, batch, cache), 1.0),), connection=self.mixer_connection)
+        if "ffn" in self.parts:
+            x, residual = self.ffn_norm.forward_streams(pending, residual, self.ffn_connection)
+            pending = Pending(((self.ffn.forward(x, batch), 1.0),), connection=self.ffn_connection)
+        return pending, residual
+
+
+CONNECTIONS.register("hyper_connection", HyperConnection)
+BLOCKS.register("hyper_connections", HyperConnectionBlock)
 BLOCKS.register("prenorm_residual", PreNormResidualBlock)
 BLOCKS.register("postnorm_residual", PostNormResidualBlock)
 BLOCKS.register("sandwich_residual", SandwichResidualBlock)

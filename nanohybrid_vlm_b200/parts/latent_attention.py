@@ -3,7 +3,9 @@
 Parameters: ``num_heads`` (H), ``head_dim`` (dn: the part of a query / key head that is not rotated), ``rot_dim`` (dr:
 the rotated part), ``v_head_dim`` (dv), ``q_rank``, ``kv_rank``, ``scale`` (on the scores), ``position`` (a PartSpec of a
 position encoding with a rotary table over at most dr elements), ``eps`` (of the two latent norms), ``sink`` (True: a
-learned number per head joins the softmax denominator), ``output_gate`` (None, or "sigmoid_head": head h's output times
+learned number per head joins the softmax denominator), ``window`` (None: all keys; n: the last n), ``rope_layout``
+("half": element i of the rotated part turns with element i + dims / 2, the default; "interleaved": element 2i with element
+2i + 1), ``output_gate`` (None, or "sigmoid_head": head h's output times
 sigmoid(g(x))_h, one number per head).
 
 With x the mixer's input:  c_q = rmsnorm(dq x) * dq.norm;  q = uq c_q, per head [dn | dr];  dkv x = [latent | key part]:
@@ -18,7 +20,7 @@ packed from the checkpoint's ``dkv`` and ``g``, ``dkv.norm`` [kv_rank], ``uk`` [
 ``sink`` [H] (float32), ``o`` [width, H dv].  Norms, rotation, scores and softmax are computed in 32-bit.
 
 Two forms of one step.  Single tokens (and float32) attend over the latents as above.  A bfloat16 step with prompt
-portions expands the latents of its requests into keys [uk_h c | k_r] and values uv_h c per head, padded to a common
+portions expands the latents of its requests (those that its tokens see) into keys [uk_h c | k_r] and values uv_h c per head, padded to a common
 head size D, in temporary pages, and runs the tensor-core attention kernels over those: a query then costs
 dn + dr + dv operations per key and head instead of 2 kv_rank + dr, and the expansion is one product over the
 requests' tokens.  The two forms differ by rounding only (which of the factors is rounded to bfloat16 on the way).
@@ -44,6 +46,12 @@ class LatentAttention(Mixer):
         self.gate = spec.get("output_gate")
         if self.gate not in (None, "sigmoid_head"):
             raise ValueError(f"an output gate is None or 'sigmoid_head', not {self.gate!r}")
+        self.window = spec.get("window")
+        if self.window is not None and int(self.window) <= 0:
+            raise ValueError("latent attention: a window must be positive")
+        self.rope_layout = spec.get("rope_layout", "half")
+        if self.rope_layout not in ("half", "interleaved"):
+            raise ValueError(f"unknown rope_layout {self.rope_layout!r}")
         self.position = env.position(spec.get("position"))
         if min(self.H, self.dn + self.dr, self.dv, self.q_rank, self.rank) <= 0 or self.dn < 0 or self.dr < 0:
             raise ValueError("latent attention: sizes must be positive")
@@ -78,7 +86,7 @@ class LatentAttention(Mixer):
             self.ukv = torch.cat([self.w_uk, self.w_uv]).contiguous()
 
     def cache_need(self):
-        return PagedKVNeed(1, self.row, v_head_dim=self.rank, planes=1)
+        return PagedKVNeed(1, self.row, self.window, v_head_dim=self.rank, planes=1)
 
     def streamed_weights(self):
         return [(self.w_dq, 0), (self.w_uq, 0), (self.w_dkvg, 0), (self.w_o, 0)]
@@ -98,7 +106,7 @@ class LatentAttention(Mixer):
         q_lat = self.new(T, H * self.row)
         ops.latent_rope_store(kvg[:, :self.row], q, q_lat, cache.pages if cache.writes else None,
                               cache.tables.slot_mapping, batch.positions, table, rotary_dim, H, self.dn, self.dr,
-                              self.rank, self.eps, self.w_dkv_norm)
+                              self.rank, self.eps, self.w_dkv_norm, interleaved=self.rope_layout == "interleaved")
         gate = kvg[:, self.row:] if self.gate else None
         if (self.ukv is not None and EXPAND_PROMPT_PORTIONS and batch.n_prefill_tokens > 0
                 and attention_mma.supports(self.D, H, H, batch.n_seqs)):
@@ -110,7 +118,7 @@ class LatentAttention(Mixer):
             q_lat.view(T, H, self.row)[:, :, :self.rank].zero_()
         o_lat = self.new(T, H * self.rank)
         ops.latent_attention(o_lat, q_lat, cache.pages, cache.tables, batch, H, self.rank, self.row, self.scale,
-                             self.w_sink if self.has_sink else None)
+                             self.w_sink if self.has_sink else None, self.window or 0)
         o = self.new(T, H * self.dv)
         ops.linear_heads(o.view(T, H, self.dv), o_lat.view(T, H, self.rank), self.uv_heads)
         if self.gate:
@@ -124,15 +132,15 @@ class LatentAttention(Mixer):
         their single tokens ride along)."""
         T, H, D = q.shape[0], self.H, self.D
         qp, pages, tables = ops.latent_expand(cache.pages, cache.tables, batch, q, q_lat, self.ukv, H, self.dn, self.dr,
-                                              self.dv, self.rank, D)
+                                              self.dv, self.rank, D, self.window or 0)
         padded = self.new(T, H * D)
         ops.attention_tensor_core(padded, qp, pages, tables, batch.cu_q, batch.kv_len, batch.n_seqs,
                                   batch.n_prefill_tokens, batch.n_prefill_seqs, batch.n_decode_seqs, batch.max_kv_len, H, H,
-                                  D, self.scale, 0, self.w_sink if self.has_sink else None)
-        o = self.new(T, H * self.dv)
+                                  D, self.scale, self.window or 0, self.w_sink if self.has_sink else None)
+        o = padded if D == self.dv and not self.gate else self.new(T, H * self.dv)
         if self.gate:
             ops.sigmoid_mul_heads(o, padded, gate, self.dv, x_head=D)
-        else:
+        elif o is not padded:
             o.view(T, H, self.dv).copy_(padded.view(T, H, D)[:, :, :self.dv])
         y = self.new(T, self.env.hidden_size)
         ops.linear(y, o, self.w_o)

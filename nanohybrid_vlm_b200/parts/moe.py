@@ -15,7 +15,10 @@ the shared output is multiplied by sigmoid(sg(x)), one number per token, ``share
 ("softmax", the default, or "sigmoid": each output's score is the sigmoid of its own logit), ``renorm`` (True: the chosen
 scores are divided by their sum; False: they are the weights as they are), ``weight_on`` ("output", the default: a
 chosen expert's output is multiplied by its weight; "input": its input is, out = sum of expert(w * x)), ``limit`` None
-(no clamp) and ``up_shift`` (what is added to the up half, 1 unless given): limit None, alpha 1, up_shift 0 make the
+(no clamp), ``scores`` "chosen_softmax" (the choice is by the logits plus, with ``correction``, a bias, and the weights
+are the softmax of these over the chosen alone), ``correction_source`` (the checkpoint's name of the correction, default
+"correction"), ``unit`` ("glu", the default, or "relu2": experts without a gate, down(relu(up x)^2), and no ``gate``
+tensors) and ``up_shift`` (what is added to the up half, 1 unless given): limit None, alpha 1, up_shift 0 make the
 experts plain gated units, down(silu(gate x) * (up x)).
 
 Router: z = router(x) with 32-bit sums; s = softmax(z) over all outputs; choice by s + correction; the weights of the
@@ -87,8 +90,11 @@ class RoutedMoE(FeedForward):
         self.scores = spec.get("scores", "softmax")
         self.renorm = bool(spec.get("renorm", True))
         self.weight_on = spec.get("weight_on", "output")
-        if self.scores not in ("softmax", "sigmoid") or self.weight_on not in ("output", "input"):
-            raise ValueError(f"unknown router scores {self.scores!r} or weight_on {self.weight_on!r}")
+        self.unit = spec.get("unit", "glu")
+        self.correction_source = spec.get("correction_source", "correction")
+        if (self.scores not in ("softmax", "sigmoid", "chosen_softmax") or self.weight_on not in ("output", "input")
+                or self.unit not in ("glu", "relu2")):
+            raise ValueError(f"unknown router scores {self.scores!r}, weight_on {self.weight_on!r} or unit {self.unit!r}")
         if self.weight_on == "input" and self.I0:
             raise ValueError("identity experts are not offered with weights on the experts' inputs")
         self.has_correction = bool(spec.get("correction", True))
@@ -109,9 +115,11 @@ class RoutedMoE(FeedForward):
             router.append(Source(self.SHARED_PREFIX + "sg", self.N, 1))
         decls = [ParamDecl("router", (self.N + int(self.shared_gate), W), sources=tuple(router))]
         if self.has_correction:
-            decls.append(ParamDecl("correction", (self.N,), init="zeros_noise", storage="float32"))
+            decls.append(ParamDecl("correction", (self.N,), init="zeros_noise", storage="float32",
+                                   sources=(Source(self.correction_source, 0, self.N),)))
+        if self.unit == "glu":
+            decls.append(ParamDecl("gate", (E, I, W), sources=tuple(Source(f"e{j}.gate", j, 1, squeeze=True) for j in range(E))))
         decls += [
-            ParamDecl("gate", (E, I, W), sources=tuple(Source(f"e{j}.gate", j, 1, squeeze=True) for j in range(E))),
             ParamDecl("up", (E, I, W), sources=tuple(Source(f"e{j}.up", j, 1, squeeze=True) for j in range(E))),
             ParamDecl("down", (E, W, I), sources=tuple(Source(f"e{j}.down", j, 1, squeeze=True) for j in range(E))),
         ]
@@ -140,7 +148,7 @@ class RoutedMoE(FeedForward):
                       scores=self.scores, renorm=self.renorm)
         on_input = self.weight_on == "input"
         # a weight on an expert's input is a factor on the 32-bit sums of its two first products
-        y, slot_pos = ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, ids, self.limit, self.alpha, self.up_shift,
+        y, slot_pos = ops.moe_experts(x, self.w_gate if self.unit == "glu" else None, self.w_up, self.w_down, ids, self.limit, self.alpha, self.up_shift,
                                       weights if on_input else None)
         shared = self.shared.forward(x, batch) if self.shared is not None else None
         out = self.new(T, W)

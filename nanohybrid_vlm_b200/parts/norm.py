@@ -1,11 +1,15 @@
 """Norms: RMSNorm with the residual add fused in (nanovllm/layers/layernorm.py:5-50), and Dynamic Tanh.
 
 Parameters: ``width``, ``eps``, ``weight_offset`` (0 for ``x * w``; 1 for the ``x * (1 + w)``
-convention some models store), ``source`` (the checkpoint's name of the weight, default "weight"), ``groups`` (the
+convention some models store), ``source`` (the checkpoint's name of the weight, default "weight"), ``own_name`` (True: the
+part's tensor carries that name too, so that several norms can share a layer's prefix), ``groups`` (the
 row is cut into this many equal consecutive parts and each is divided by the root mean square of its own elements;
 default 1; over a float32 stream only), ``post_scale`` (the checkpoint's name of a second vector [width] that multiplies
 the normed output after the weight, a scale per channel on a sub-block's contribution; only where the norm adds a
 sub-block's output onto a float32 stream, ``add_normed``).
+
+Over a residual stream of several copies (``forward_streams``, and ``forward_add_rows`` given a :class:`Pending` with a
+connection) one kernel rebuilds the copies from the pending output, sums what the next sub-block reads and norms it.
 
 Over a residual stream kept in float32 (``forward_add`` / ``forward_add_rows`` given a :class:`Pending`) the terms
 are added in 32-bit, the statistics and the product with the weight are 32-bit, and the result is rounded once.
@@ -30,6 +34,8 @@ class RMSNorm(Norm):
         if self.groups < 1 or self.width % self.groups:
             raise ValueError(f"a norm over {self.width} elements does not divide into {self.groups} parts")
         self.post_scale = spec.get("post_scale")
+        # the part's tensor: with a scale beside it, or on request, it carries the checkpoint's name
+        self.local = self.source if self.post_scale is not None or spec.get("own_name") else "weight"
 
     def _plain_only(self):
         if self.groups != 1:
@@ -38,10 +44,7 @@ class RMSNorm(Norm):
             raise TypeError("a norm with a scale per channel adds a sub-block's output onto a float32 stream (add_normed)")
 
     def params(self):
-        # the tensors carry the checkpoint's names where a scale comes with the norm, so that two such norms can share
-        # a layer's prefix
-        name = "weight" if self.post_scale is None else self.source
-        decls = [ParamDecl(name, (self.width,), init="norm" if self.weight_offset == 0.0 else "zeros_noise",
+        decls = [ParamDecl(self.local, (self.width,), init="norm" if self.weight_offset == 0.0 else "zeros_noise",
                            sources=(Source(self.source, 0, self.width),))]
         if self.post_scale is not None:
             decls.append(ParamDecl(self.post_scale, (self.width,), init="layer_scale",
@@ -49,9 +52,9 @@ class RMSNorm(Norm):
         return decls
 
     def bind(self, tensors):
-        if self.post_scale is None:
-            return super().bind(tensors)
-        self.w_weight, self.w_post_scale = tensors[self.source], tensors[self.post_scale]
+        self.w_weight = tensors[self.local]
+        if self.post_scale is not None:
+            self.w_post_scale = tensors[self.post_scale]
 
     def add_normed(self, terms, residual, side_eps=None, want_rounded=True):
         if self.groups != 1 or self.weight_offset != 0.0:
@@ -59,6 +62,27 @@ class RMSNorm(Norm):
         rounded = self.new(*residual.shape) if want_rounded else None
         ops.postnorm_stream(residual, rounded, terms, self.w_weight, getattr(self, "w_post_scale", None), self.eps, side_eps)
         return rounded
+
+    def _streams(self, x, streams, n_streams, read, dst, rows):
+        if self.groups != 1 or self.weight_offset != 0.0 or self.post_scale is not None:
+            raise TypeError("over several streams the norm is a plain RMS norm (one group, the weight as it is stored)")
+        y, con = None, x.connection
+        if x.terms:
+            if con is None or x.post is not None or len(x.terms) > 1 or x.terms[0][1] != 1.0:
+                raise TypeError("over several streams one output is pending at most, with factor 1 and a connection")
+            y = x.terms[0][0]
+        out = self.new(streams.shape[0] if rows is None else rows.numel(), self.width)
+        ops.streams_rmsnorm(out, dst, streams, self.w_weight, self.eps, y, con.mix if y is not None else None,
+                            con.write if y is not None else None, read, rows, n_streams)
+        return out
+
+    def forward_streams(self, x, streams, connection):
+        S = connection.streams
+        if not x.terms:
+            return self._streams(x, streams, S, connection.read, None, None), streams
+        # the first output that joins makes the copies; from then on they are rebuilt in place
+        new = streams if streams.shape[1] == S else self.new(streams.shape[0], S, self.width, dtype=torch.float32)
+        return self._streams(x, streams, S, connection.read, new, None), new
 
     def forward(self, x):
         self._plain_only()
@@ -81,6 +105,8 @@ class RMSNorm(Norm):
         return out
 
     def forward_add_rows(self, x, residual, rows):
+        if isinstance(x, Pending) and x.connection is not None:      # the norm of the sum of the new copies
+            return self._streams(x, residual, x.connection.streams, None, None, rows)
         if isinstance(x, Pending):
             x = x.settled()
             out = self.new(rows.numel(), residual.shape[-1])

@@ -23,13 +23,19 @@ positions, and their pages are kept), ``sink_constant`` (a number: the denominat
 learned sink would, but no tensor is read; 0.0 adds one), ``qk_norm_order`` ("after_rotation", the default, or
 "before_rotation": the unit norm and its weight come before the rotation), ``rope_layout`` ("half": element i turns
 with element i + dims / 2, the default; "interleaved": element 2i with element 2i + 1), ``bias`` may also be "qk":
-biases on q and k only.
+biases on q and k only, ``qk_norm_scope`` ("head", the default, or "projection": all query heads are divided by ONE root
+mean square over the whole query projection, the key heads likewise, and the weights ``q.norm`` / ``k.norm`` have that
+size; before the rotation, with a weight), ``value_mix`` (None; "source": the layer leaves its values to the later layers
+of the step; "mixed": the values become (1 - lambda) v + lambda v_source of the same token, lambda a learned number
+``vmix``, and the mixed values are what the pages keep; with ``qk_norm_scope`` "projection" only).
 
 Tensors: ``qkv`` [(nq + nkv) d (+ nkv dv) (+ nq dv), width], rows q then k then v then g, packed from the
 checkpoint's ``q``, ``k``, ``v``, ``g`` (those that exist); ``qk_bias`` [(nq + nkv) d] from ``q.b``, ``k.b``; ``sink``
 [nq] (float32); ``o`` [width, nq dv]; ``o.b`` [width].  Scores, softmax, rotation, bias and norm are computed in 32-bit.
 """
 from __future__ import annotations
+
+import torch
 
 from ..kernels import ops
 from .base import MIXERS, Mixer, PagedKVNeed
@@ -54,11 +60,14 @@ class SinkAttention(Mixer):
         if self.sink_constant is not None:
             if spec.get("sink", False):
                 raise ValueError("a sink is learned (sink=True) or a constant (sink_constant), not both")
-            import torch
             self.has_sink = False
             self.fixed_sinks = torch.full((self.nq,), float(self.sink_constant), dtype=torch.float32, device=env.device)
         self.keep_first = int(spec.get("keep_first", 0) or 0)
-        self.norm_order = spec.get("qk_norm_order", "after_rotation")
+        self.norm_scope = spec.get("qk_norm_scope", "head")
+        self.value_mix = spec.get("value_mix")
+        if self.norm_scope not in ("head", "projection") or self.value_mix not in (None, "source", "mixed"):
+            raise ValueError(f"unknown qk_norm_scope {self.norm_scope!r} or value_mix {self.value_mix!r}")
+        self.norm_order = spec.get("qk_norm_order", "before_rotation" if self.norm_scope == "projection" else "after_rotation")
         self.rope_layout = spec.get("rope_layout", "half")
         if self.norm_order not in ("after_rotation", "before_rotation") or self.rope_layout not in ("half", "interleaved"):
             raise ValueError(f"unknown qk_norm_order {self.norm_order!r} or rope_layout {self.rope_layout!r}")
@@ -87,9 +96,19 @@ class SinkAttention(Mixer):
         base = spec.get("distance_slope_base")
         self.slopes = None
         if base is not None:
-            import torch
             self.slopes = torch.tensor([2.0 ** (-float(base) * (h + 1) / self.nq) for h in range(self.nq)],
                                        dtype=torch.float32, device=env.device)
+        self.rows = self.norm_scope == "projection"         # q and k pass the kernel that works on a token's whole rows
+        if self.rows and (not self.norm_weight or self.norm_order != "before_rotation" or self.bias or not self.own_kv
+                          or self.values != "projected"):
+            raise ValueError("a norm over the whole projection has a weight, comes before the rotation and goes with keys "
+                             "and values of the layer's own, without biases")
+        if self.value_mix and not self.rows:
+            raise ValueError("mixed values are offered with a norm over the whole projection")
+        # what a page row and a query head hold: on the tensor cores keys and values of unequal size are padded to one
+        self.D = self.d
+        if self.rows and env.dtype == torch.bfloat16 and (self.dv > self.d or self.d % 16):
+            self.D = -(-max(self.d, self.dv) // 16) * 16
         self.q_size = self.nq * self.d
         self.k_size = self.nkv * self.d if self.own_kv else 0
         self.v_size = self.nkv * self.dv if self.values == "projected" and self.own_kv else 0
@@ -111,9 +130,11 @@ class SinkAttention(Mixer):
         if self.has_sink:
             decls.append(ParamDecl("sink", (self.nq,), storage="float32"))
         if self.norm_weight:
-            decls.append(ParamDecl("q.norm", (self.d,), init="norm"))
+            decls.append(ParamDecl("q.norm", (self.q_size if self.rows else self.d,), init="norm"))
             if self.own_kv:
-                decls.append(ParamDecl("k.norm", (self.d,), init="norm"))
+                decls.append(ParamDecl("k.norm", (self.k_size if self.rows else self.d,), init="norm"))
+        if self.value_mix == "mixed":
+            decls.append(ParamDecl("vmix", (1,), init="mix_share", storage="float32", sources=(Source("vmix", 0, 1, squeeze=True),)))
         if self.bias:
             if not self.own_kv:
                 raise ValueError("projection biases are not offered for a layer without keys of its own")
@@ -124,7 +145,7 @@ class SinkAttention(Mixer):
         return decls
 
     def cache_need(self):
-        return PagedKVNeed(self.nkv, self.d, self.keep_window, v_head_dim=self.dv, chunk=self.chunk,
+        return PagedKVNeed(self.nkv, self.D, self.keep_window, v_head_dim=self.dv, chunk=self.chunk,
                            keep_first=self.keep_first)
 
     def streamed_weights(self):
@@ -136,17 +157,21 @@ class SinkAttention(Mixer):
         ops.linear(qkv, x, self.w_qkv)
         rot = self.position.rotary() if self.position is not None else None
         table, rotary_dim = rot if rot is not None else (None, 0)
-        q = self.new(T, self.q_size)
+        q = self.new(T, self.nq * self.D)
         if cache.writes != self.own_kv:
             raise ValueError("a layer with keys of its own writes its pages; one without reads another run's (cache_from)")
-        ops.rope_norm_store(qkv, q, cache.pages if cache.writes else None, cache.tables.slot_mapping, batch.positions,
-                            table, rotary_dim, self.nq, self.nkv, self.d, self.dv, self.eps,
-                            bias=self.w_qk_bias if self.bias else None, values_from_keys=self.values == "keys",
-                            q_weight=self.w_q_norm if self.norm_weight else None,
-                            k_weight=self.w_k_norm if self.norm_weight and self.own_kv else None,
-                            norm_first=self.norm_order == "before_rotation", interleaved=self.rope_layout == "interleaved")
+        if self.rows:
+            self._store_rows(qkv, q, batch, cache, table, rotary_dim)
+        else:
+            ops.rope_norm_store(qkv, q, cache.pages if cache.writes else None, cache.tables.slot_mapping, batch.positions,
+                                table, rotary_dim, self.nq, self.nkv, self.d, self.dv, self.eps,
+                                bias=self.w_qk_bias if self.bias else None, values_from_keys=self.values == "keys",
+                                q_weight=self.w_q_norm if self.norm_weight else None,
+                                k_weight=self.w_k_norm if self.norm_weight and self.own_kv else None,
+                                norm_first=self.norm_order == "before_rotation",
+                                interleaved=self.rope_layout == "interleaved")
         o = self.new(T, self.nq * self.dv)
-        ops.attention_sink(o, q, cache.pages, cache.tables, batch, self.nq, self.nkv, self.d, self.dv, self.scale,
+        ops.attention_sink(o, q, cache.pages, cache.tables, batch, self.nq, self.nkv, self.D, self.dv, self.scale,
                            self.w_sink if self.has_sink else getattr(self, "fixed_sinks", None), self.window or 0,
                            self.chunk or 0, self.slopes, self.keep_first)
         if self.gate == "sigmoid_head":
@@ -158,6 +183,21 @@ class SinkAttention(Mixer):
         if self.out_bias:
             ops.add_row_bias(y, self.w_o_b)
         return y
+
+    VALUE_SOURCE = "value_source"       # the key under which a step carries the values that later layers mix in
+
+    def _store_rows(self, qkv, q, batch, cache, table, rotary_dim):
+        v_first = share = None
+        v = qkv[:, self.q_size + self.k_size:self.q_size + self.k_size + self.v_size]
+        if self.value_mix == "source":
+            batch.carried[self.VALUE_SOURCE] = v
+        elif self.value_mix == "mixed":
+            v_first, share = batch.carried.get(self.VALUE_SOURCE), self.w_vmix
+            if v_first is None or v_first.shape != v.shape:
+                raise ValueError("a layer that mixes values needs an earlier layer of the step that leaves values of its size")
+        ops.row_norm_store(qkv, q, self.D, cache.pages, cache.tables.slot_mapping, batch.positions, table, rotary_dim,
+                           self.nq, self.nkv, self.d, self.dv, self.eps, self.w_q_norm, self.w_k_norm,
+                           interleaved=self.rope_layout == "interleaved", v_first=v_first, v_share=share)
 
 
 MIXERS.register("sink_attention", SinkAttention)
