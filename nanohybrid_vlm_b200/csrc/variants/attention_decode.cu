@@ -1,5 +1,7 @@
 // bfloat16 attention of single decoded tokens over cache pages, for head sizes in steps of 64 and pages that are a
-// multiple of 32 keys; compiled once per head size (-DNHV_ATTN_D=<head size>).  Replaces the library call at
+// multiple of 32 keys; compiled once per head size (-DNHV_ATTN_D=<head size>), and per size of a value head where that
+// is smaller (-DNHV_ATTN_DV, a multiple of 64; page rows stay D wide, of a value row only the first DV elements are read).
+//  Replaces the library call at
 // nanovllm/layers/attention.py:72-74 (flash_attn_with_kvcache).
 //
 // Decoding reads every key and value of every live request once and computes almost nothing, so the kernel is built
@@ -58,17 +60,22 @@
 #error "compile with -DNHV_ATTN_D=<head size>"
 #endif
 
+#ifndef NHV_ATTN_DV
+#define NHV_ATTN_DV NHV_ATTN_D
+#endif
+
 namespace {
 
-constexpr int D = NHV_ATTN_D;
+constexpr int D = NHV_ATTN_D, DV = NHV_ATTN_DV;
 static_assert(D % 64 == 0 && D >= 64 && D <= 256, "head sizes 64, 128, 192 and 256");
-constexpr int CH = D / 8;          // 16-byte chunks in a row
-constexpr int DB = D / 64;         // 128-byte column blocks of a head (one TMA box each)
+static_assert(DV % 64 == 0 && DV >= 64 && DV <= D, "value heads are a multiple of 64 up to the head size");
+constexpr int CH = D / 8, CHV = DV / 8;    // 16-byte chunks in a row of keys, of values
+constexpr int DB = D / 64, VB = DV / 64;   // 128-byte column blocks of a head (one TMA box each)
 constexpr int BN = 32;             // keys per tile
 constexpr int KS = D / 16;         // k-steps of Q.K^T
-constexpr int DN = D / 8;          // n-tiles of P.V
-constexpr int TILE_BYTES = BN * D * 2;                 // one K tile or one V tile
-constexpr int STAGE_BYTES = 2 * TILE_BYTES;
+constexpr int DN = DV / 8;         // n-tiles of P.V
+constexpr int TILE_BYTES = BN * D * 2;                 // one K tile
+constexpr int STAGE_BYTES = TILE_BYTES + BN * DV * 2;  // and its V tile
 // Consumer warps and ring stages.  A stage is always consumed by the same warp (STAGES is a multiple of NCW and
 // tile number t of the block goes to warp t % NCW and stage t % STAGES): a warp's waits on one barrier then follow
 // one another, so it can never ask for a phase while the one before it is still filling (a wait by parity cannot
@@ -79,7 +86,7 @@ constexpr int STAGES_MIN = 2 * NCW;
 constexpr int STAGES_DEEP = D <= 128 ? 3 * NCW : STAGES_MIN;
 constexpr int THREADS = (NCW + 1) * 32;
 constexpr int Q_BYTES = 16 * D * 2;
-constexpr int merge_bytes(int mrows) { return NCW * mrows * D * 4 + NCW * mrows * 2 * 4; }
+constexpr int merge_bytes(int mrows) { return NCW * mrows * DV * 4 + NCW * mrows * 2 * 4; }
 constexpr int MAX_SEQS = 512;
 constexpr size_t smem_bytes(int stages, int mrows) { return 1024 + (size_t)stages * STAGE_BYTES + merge_bytes(mrows) + Q_BYTES; }
 // what the kernel declares beside that: the new key and value, the rows copied ahead, the plan's numbers per request
@@ -278,6 +285,7 @@ __device__ __forceinline__ void warp_half_tile(RowState& st, const uint32_t (&qf
 }
 
 struct alignas(64) Params {
+  CUtensorMap v_map;        // value heads smaller than the key heads: a box is a tile's values alone (pool_map: its keys)
   CUtensorMap pool_map;     // the pool in four dimensions: one box is a tile's keys and values (see where it is made)
   const bf16* q;            // plain form: [tokens, nq * D]
   bf16* out;
@@ -285,11 +293,12 @@ struct alignas(64) Params {
   const int* block_table;
   const int* cu_q;
   const int* kv_len;
-  float* part_o;            // [grid][2][16][D]
+  float* part_o;            // [grid][2][16][DV]
   float* part_ml;           // [grid][2][16][2]
   int* counters;            // [n_seqs * head_blocks], zero; left zero
   const float* sinks;       // per query head, or null: exp(sink) joins the softmax denominator once, where a head's sum is final
   int q_stride, out_stride, bt_stride, n_seqs, nq, nkv, page_size, n_pages, window, chunk;
+  int out_head;             // elements between two heads of the output, up to DV: that many are written
   int keep_first;           // with a window: the keys at positions below it stay visible; their tiles come first
   float scale_log2;
   FusedQK fq;
@@ -308,8 +317,8 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
   extern __shared__ unsigned char smem_unaligned[];
   unsigned char* smem = smem_unaligned + ((1024 - (smem_u32(smem_unaligned) & 1023)) & 1023);
   unsigned char* ring = smem;                                                   // [STAGES][K tile | V tile]
-  float* mo = reinterpret_cast<float*>(smem + (size_t)STAGES * STAGE_BYTES);    // [NCW][MROWS][D]
-  float* mml = mo + NCW * MROWS * D;                                            // [NCW][MROWS][2]
+  float* mo = reinterpret_cast<float*>(smem + (size_t)STAGES * STAGE_BYTES);    // [NCW][MROWS][DV]
+  float* mml = mo + NCW * MROWS * DV;                                           // [NCW][MROWS][2]
   bf16* qbuf = reinterpret_cast<bf16*>(mml + NCW * MROWS * 2);                  // [16][D], chunks exchanged as in a tile
   __shared__ __align__(16) bf16 s_new[2][D];                  // the new token's key and value (fused form)
   // fused form: the rows of qkv that the piece after the one at work needs, as they lie in qkv (the head block's
@@ -404,7 +413,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
     for (int sq = c; sq < n_seqs; sq += gridDim.x) {
       if (!s_idle[sq]) continue;
       bf16* dst = p.out + (size_t)s_tok[sq] * p.out_stride;
-      for (int id = tid; id < p.nq * CH; id += n_threads) reinterpret_cast<uint4*>(dst)[id] = make_uint4(0, 0, 0, 0);
+      for (int id = tid; id < p.nq * (p.out_head / 8); id += n_threads) reinterpret_cast<uint4*>(dst)[id] = make_uint4(0, 0, 0, 0);
     }
   };
   if (c >= NB || T == 0) {
@@ -500,6 +509,9 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
           // the whole tile in one copy: the box holds 64 columns x the tile's keys x the head's column blocks x
           // (keys, values), and arrives in that order (a copy costs the TMA unit about as much whatever it holds)
           if (lane == 0) tma_load_4d(ring + (size_t)stage * STAGE_BYTES, &p.pool_map, 0, rk, 0, 0, &full[stage]);
+          if constexpr (DV < D) {                            // narrower values: a copy of their own
+            if (lane == 0) tma_load_4d(ring + (size_t)stage * STAGE_BYTES + TILE_BYTES, &p.v_map, 0, rk, 0, 1, &full[stage]);
+          }
           ++gi;
         }
       }
@@ -648,8 +660,8 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
       const int r_hi = there ? min(BN, max(0, total - key_base)) : BN;         // rows [r_hi, BN) are beyond it
       const int r_keep = there ? min(BN, max(0, keep_first - key_base)) : 0;   // rows [0, r_keep) are kept first keys
       if (r_lo > r_keep || r_hi < BN) {
-        for (int id = lane; id < BN * CH; id += 32) {
-          const int r = id / CH, cc = id - r * CH;
+        for (int id = lane; id < BN * CHV; id += 32) {
+          const int r = id / CHV, cc = id - r * CHV;
           if ((r < r_lo && r >= r_keep) || r >= r_hi) *reinterpret_cast<uint4*>(vt + tile_off<BN>(r, cc)) = make_uint4(0, 0, 0, 0);
         }
         wrote = true;
@@ -672,7 +684,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
       l += __shfl_xor_sync(0xffffffffu, l, 2);
       const int R = (lane >> 2) + 8 * i;
       if (R >= gn) continue;                                   // rows beyond the group hold nothing
-      float* dst = mo + ((size_t)warp * MROWS + R) * D + ((lane & 3) << 1);
+      float* dst = mo + ((size_t)warp * MROWS + R) * DV + ((lane & 3) << 1);
 #pragma unroll
       for (int n = 0; n < DN; ++n)
         *reinterpret_cast<float2*>(dst + n * 8) = make_float2(st.o[n][2 * i], st.o[n][2 * i + 1]);
@@ -686,10 +698,10 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
     // a block has at most two pieces that are not whole: one that goes on where the block before it stopped (only
     // at the start of its range) and one that its range's end cuts short (only at that end)
     const int slot = pc.t_begin > 0 ? 0 : 1;
-    float* po = p.part_o + ((size_t)c * 2 + slot) * 16 * D;
+    float* po = p.part_o + ((size_t)c * 2 + slot) * 16 * DV;
     float* pml = p.part_ml + ((size_t)c * 2 + slot) * 16 * 2;
-    for (int id = threadIdx.x; id < gn * (D / 4); id += NCW * 32) {
-      const int R = id / (D / 4), c4 = id - R * (D / 4);
+    for (int id = threadIdx.x; id < gn * (DV / 4); id += NCW * 32) {
+      const int R = id / (DV / 4), c4 = id - R * (DV / 4);
       float M = -INFINITY;
 #pragma unroll
       for (int w = 0; w < NCW; ++w) M = fmaxf(M, mml[(w * MROWS + R) * 2]);
@@ -699,17 +711,17 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
       for (int w = 0; w < NCW; ++w) {
         const float mw = mml[(w * MROWS + R) * 2];
         const float f = mw == -INFINITY ? 0.f : exp2f(mw - M);
-        const float4 t = *reinterpret_cast<const float4*>(mo + ((size_t)w * MROWS + R) * D + c4 * 4);
+        const float4 t = *reinterpret_cast<const float4*>(mo + ((size_t)w * MROWS + R) * DV + c4 * 4);
         acc.x += t.x * f; acc.y += t.y * f; acc.z += t.z * f; acc.w += t.w * f;
         L += mml[(w * MROWS + R) * 2 + 1] * f;
       }
       if (whole) {
         if (p.sinks && L > 0.f) L += exp2f(fmaf(p.sinks[kvh * G + g0 + R], LOG2E, -M));
         const float inv = L > 0.f ? 1.0f / L : 0.f;
-        bf16* dst = p.out + tok * p.out_stride + (size_t)(kvh * G + g0 + R) * D + c4 * 4;
-        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
+        bf16* dst = p.out + tok * p.out_stride + (size_t)(kvh * G + g0 + R) * p.out_head + c4 * 4;
+        if (c4 * 4 < p.out_head) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
       } else {
-        *reinterpret_cast<float4*>(po + R * D + c4 * 4) = acc;
+        *reinterpret_cast<float4*>(po + R * DV + c4 * 4) = acc;
         if (c4 == 0) { pml[R * 2] = M; pml[R * 2 + 1] = L; }
       }
     }
@@ -729,8 +741,8 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
         // the first owner's piece starts with the first tile (slot 1); every other owner's goes on from the block
         // before it (slot 0)
         constexpr int first_slot = 1;
-        for (int id = threadIdx.x; id < gn * (D / 4); id += NCW * 32) {
-          const int R = id / (D / 4), c4 = id - R * (D / 4);
+        for (int id = threadIdx.x; id < gn * (DV / 4); id += NCW * 32) {
+          const int R = id / (DV / 4), c4 = id - R * (DV / 4);
           // One pass, eight pieces' loads on their way at a time (the pieces lie in L2: what this costs is trips,
           // not bytes): the running maximum moves with every eight, and what is summed so far is rescaled to it.
           float M = -INFINITY, L = 0.f;
@@ -742,7 +754,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
             for (int j = 0; j < 8; ++j) {
               const int k = min(k0 + j, pieces - 1);
               const size_t at = ((size_t)(first_owner + k) * 2 + (k == 0 ? first_slot : 0)) * 16;
-              t[j] = __ldcg(reinterpret_cast<const float4*>(p.part_o + (at + R) * D) + c4);
+              t[j] = __ldcg(reinterpret_cast<const float4*>(p.part_o + (at + R) * DV) + c4);
               ml[j] = __ldcg(reinterpret_cast<const float2*>(p.part_ml + (at + R) * 2));     // (max, sum)
             }
             float Mb = M;
@@ -764,8 +776,8 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
           }
           if (p.sinks && L > 0.f) L += exp2f(fmaf(p.sinks[kvh * G + g0 + R], LOG2E, -M));
           const float inv = L > 0.f ? 1.0f / L : 0.f;
-          bf16* dst = p.out + tok * p.out_stride + (size_t)(kvh * G + g0 + R) * D + c4 * 4;
-          *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
+          bf16* dst = p.out + tok * p.out_stride + (size_t)(kvh * G + g0 + R) * p.out_head + c4 * 4;
+          if (c4 * 4 < p.out_head) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
         }
         if (threadIdx.x == 0) p.counters[unit] = 0;            // ready for the next launch
       }
@@ -801,7 +813,7 @@ NHV_API void* NHV_FN(nhv_attn_decode_error_word_d)() { return nhv_wait_error_add
 // The most requests one launch plans for.
 NHV_API int NHV_FN(nhv_attn_decode_max_seqs_d)() { return MAX_SEQS; }
 
-// The grid (one block per SM) and the scratch a launch needs: part_o [blocks * 2 * 16 * D] floats, part_ml
+// The grid (one block per SM) and the scratch a launch needs: part_o [blocks * 2 * 16 * DV] floats, part_ml
 // [blocks * 2 * 16 * 2] floats, and counters [n_seqs * kv_heads * ceil(group / 16)] ints that are zero (the kernel
 // leaves them zero).
 NHV_API int NHV_FN(nhv_attn_decode_blocks_d)() {
@@ -825,7 +837,10 @@ NHV_API int NHV_FN(nhv_attn_decode_d)(const void* q, int q_stride, const void* q
                                       int window, int chunk, float scale, float* part_o, float* part_ml, int* counters,
                                       const void* q_w, const void* k_w, const float* cos_sin, const int* positions,
                                       const int* slot_mapping, int rotary_dim, int max_position, int store, float eps,
-                                      float weight_offset, const float* sinks, int keep_first, cudaStream_t stream) {
+                                      float weight_offset, const float* sinks, int keep_first, int out_head, cudaStream_t stream) {
+  ATT_REQUIRE(out_head > 0 && out_head <= DV && out_head % 8 == 0,
+              "attention (decode, TMA): an output head has %d elements, in steps of 8 up to %d", out_head, DV);
+  ATT_REQUIRE(!qkv || (DV == D && out_head == D), "attention: the form that works from the projection has heads of one size");
   ATT_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention: kept first keys go with a window");
   ATT_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention: %d query heads do not divide into %d KV heads", nq, nkv);
   ATT_REQUIRE(page_size > 0 && page_size % BN == 0 && n_pages > 0 && bt_stride > 0,
@@ -860,24 +875,26 @@ NHV_API int NHV_FN(nhv_attn_decode_d)(const void* q, int q_stride, const void* q
     ATT_REQUIRE(q && q_stride % 8 == 0 && ((uintptr_t)q % 16) == 0, "attention: q must be 16-byte aligned");
   }
   static std::mutex mutex;
-  static std::unordered_map<const void*, std::pair<long long, CUtensorMap>> maps;   // one per cache pool: pools do not move
+  static std::unordered_map<const void*, std::pair<long long, std::pair<CUtensorMap, CUtensorMap>>> maps;   // one per cache pool: pools do not move
   const long long rows = (long long)n_pages * 2 * nkv * page_size;
   {
     std::lock_guard<std::mutex> lock(mutex);
     auto it = maps.find(kv_pages);
     if (it == maps.end() || it->second.first != rows) {
-      CUtensorMap m;
+      CUtensorMap m, mv;
       // the pool as [keys or values of a page][column block of 64][row of the pool][64 columns]: the values of a
       // (page, KV head) lie nkv * page_size rows behind its keys
       const long long half = (long long)nkv * page_size;
       const long long dims[4] = {64, rows - half, DB, 2};
       const long long strides[4] = {2, (long long)D * 2, 128, half * D * 2};
-      const int box[4] = {64, BN, DB, 2};
+      const int box[4] = {64, BN, DB, DV < D ? 1 : 2}, box_v[4] = {64, BN, VB, 1};
       ATT_REQUIRE(nhv_make_map_bf16_nd(&m, kv_pages, 4, dims, strides, box), "attention (decode, TMA): cannot encode the tensor map of the pool");
-      maps[kv_pages] = {rows, m};
+      ATT_REQUIRE(nhv_make_map_bf16_nd(&mv, kv_pages, 4, dims, strides, box_v), "attention (decode, TMA): cannot encode the tensor map of the values");
+      maps[kv_pages] = {rows, {m, mv}};
       it = maps.find(kv_pages);
     }
-    p.pool_map = it->second.second;
+    p.pool_map = it->second.second.first;
+    p.v_map = it->second.second.second;
   }
   const bool deep = nq / nkv <= 8;                           // groups of up to 8 heads: the smaller merge buffer, the deeper ring
   const size_t smem = deep ? smem_bytes(STAGES_DEEP, 8) : smem_bytes(STAGES_MIN, 16);
@@ -904,6 +921,7 @@ NHV_API int NHV_FN(nhv_attn_decode_d)(const void* q, int q_stride, const void* q
   p.part_ml = part_ml;
   p.counters = counters;
   p.sinks = sinks;
+  p.out_head = out_head;
   p.q_stride = q_stride; p.out_stride = out_stride; p.bt_stride = bt_stride; p.n_seqs = n_seqs; p.nq = nq; p.nkv = nkv;
   p.page_size = page_size; p.n_pages = n_pages; p.window = window; p.chunk = chunk; p.keep_first = keep_first;
   p.scale_log2 = scale * LOG2E;

@@ -25,12 +25,17 @@
 #ifndef NHV_ATTN_D
 #error "compile with -DNHV_ATTN_D=<head size>"
 #endif
+// Value heads may be smaller than key heads: page rows stay D wide, of a value row only the first DV elements are read.
+#ifndef NHV_ATTN_DV
+#define NHV_ATTN_DV NHV_ATTN_D
+#endif
 
 namespace {
 
-constexpr int D = NHV_ATTN_D;
+constexpr int D = NHV_ATTN_D, DV = NHV_ATTN_DV;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head size must be a multiple of 16 up to 256");
-constexpr int CH = D / 8;          // 16-byte chunks in a row
+static_assert(DV % 16 == 0 && DV >= 16 && DV <= D, "value heads are a multiple of 16 up to the head size");
+constexpr int CH = D / 8, CHV = DV / 8;    // 16-byte chunks in a row of keys, of values
 // ldmatrix reads one chunk column of 8 rows at a time: the 8 rows must fall into 8 different bank groups.
 // Rows of a multiple of 128 bytes swap chunks inside each group of 8 (chunk ^ (row & 7)); other head sizes
 // pad every row by one chunk, which makes the row stride odd.
@@ -39,7 +44,7 @@ constexpr int ROW_CH = SWIZZLE ? CH : CH + 1;
 constexpr int BN = 64;             // keys per tile
 constexpr int TILE_ELEMS = BN * ROW_CH * 8;
 constexpr int KS = D / 16;         // k-steps of Q.K^T
-constexpr int DN = D / 8;          // n-tiles of P.V
+constexpr int DN = DV / 8;         // n-tiles of P.V
 constexpr int THREADS = 128;
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -98,7 +103,7 @@ __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const PageGeom&
       const bool ok = page_ok && j >= lo && j < hi;
       const bf16* src = ok ? base + (size_t)r * D + c * 8 : g.kv_pages;
       cp_async16(ks + tile_off(r, c), src, ok);
-      cp_async16(vs + tile_off(r, c), ok ? src + v_off : src, ok);
+      if (CHV == CH || c < CHV) cp_async16(vs + tile_off(r, c), ok ? src + v_off : src, ok);
     }
     return;
   }
@@ -114,7 +119,7 @@ __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const PageGeom&
       if (ok) src = g.kv_pages + ((((size_t)pg * 2) * g.nkv + g.kvh) * g.page_size + (j - lp * g.page_size)) * D + c * 8;
     }
     cp_async16(ks + tile_off(r, c), src, ok);
-    cp_async16(vs + tile_off(r, c), ok ? src + v_off : src, ok);
+    if (CHV == CH || c < CHV) cp_async16(vs + tile_off(r, c), ok ? src + v_off : src, ok);
   }
 }
 
@@ -336,7 +341,7 @@ __global__ void __launch_bounds__(THREADS, MTW == 2 ? 2 : (D <= 128 ? 3 : 1)) at
     const bf16* __restrict__ kv_pages, const int* __restrict__ block_table, int bt_stride,
     const int* __restrict__ cu_q, const int* __restrict__ kv_len, int n_seqs, int nq, int nkv, int page_size,
     int n_pages, int window, int chunk, float scale_log2, int tokens_per_block, const float* __restrict__ sinks,
-    const float* __restrict__ slopes, int keep_first) {
+    const float* __restrict__ slopes, int keep_first, int out_head) {
   constexpr int PF_ROWS = 64 * MTW;                          // rows (token x head of the group) per block
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qbuf = reinterpret_cast<bf16*>(smem_raw);            // [PF_ROWS rows]
@@ -449,10 +454,10 @@ __global__ void __launch_bounds__(THREADS, MTW == 2 ? 2 : (D <= 128 ? 3 : 1)) at
       // a sink per query head: exp(sink) joins the sum once, in the units of the row's running maximum
       if (sinks && l > 0.f) l += exp2f(fmaf(sinks[kvh * G + g], LOG2E, -st.m[mt][i]));
       const float inv = l > 0.f ? 1.0f / l : 0.f;
-      bf16* dst = out + (size_t)(cu_q[seq] + t0 + tq) * out_stride + (size_t)(kvh * G + g) * D + ((lane & 3) << 1);
+      bf16* dst = out + (size_t)(cu_q[seq] + t0 + tq) * out_stride + (size_t)(kvh * G + g) * out_head + ((lane & 3) << 1);
 #pragma unroll
       for (int n = 0; n < DN; ++n)
-        *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(st.o[mt][n][2 * i] * inv, st.o[mt][n][2 * i + 1] * inv);
+        if (n * 8 < out_head) *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(st.o[mt][n][2 * i] * inv, st.o[mt][n][2 * i + 1] * inv);
     }
 }
 
@@ -533,7 +538,7 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
     const int* __restrict__ block_table, int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ kv_len,
     float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int n_seqs, int nq, int nkv,
     int page_size, int n_pages, int window, int chunk, float scale_log2, int max_pieces, const FusedQK fq,
-    const float* __restrict__ sinks, const float* __restrict__ slopes, int keep_first) {
+    const float* __restrict__ sinks, const float* __restrict__ slopes, int keep_first, int out_head) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* kbuf = reinterpret_cast<bf16*>(smem_raw);
   bf16* vbuf = kbuf + DSTAGES * TILE_ELEMS;
@@ -724,15 +729,15 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
     }
     cp_async_wait<0>();
     // merge the 4 warps (each saw a quarter of every tile) through shared memory
-    float* mo = reinterpret_cast<float*>(smem_raw);            // [4 warps][16 rows][D]
-    float* mml = mo + 4 * 16 * D;                              // [4][16][2]
+    float* mo = reinterpret_cast<float*>(smem_raw);            // [4 warps][16 rows][DV]
+    float* mml = mo + 4 * 16 * DV;                             // [4][16][2]
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       float l = st.l[i];
       l += __shfl_xor_sync(0xffffffffu, l, 1);
       l += __shfl_xor_sync(0xffffffffu, l, 2);
       const int R = (lane >> 2) + 8 * i;
-      float* dst = mo + ((size_t)warp * 16 + R) * D + ((lane & 3) << 1);
+      float* dst = mo + ((size_t)warp * 16 + R) * DV + ((lane & 3) << 1);
 #pragma unroll
       for (int n = 0; n < DN; ++n) {
         dst[n * 8] = st.o[n][2 * i];
@@ -751,10 +756,10 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
       pieces = tile_owner(piece_first + nt - 1, T, NB) - first_owner + 1;
       piece = min(c - first_owner, max_pieces - 1);          // never beyond the scratch, whatever the caller passed
     }
-    float* po = part_o + (unit * max_pieces + piece) * rows_per * D;
+    float* po = part_o + (unit * max_pieces + piece) * rows_per * DV;
     float* pml = part_ml + (unit * max_pieces + piece) * rows_per * 2;
-    for (int id = threadIdx.x; id < gn * D; id += THREADS) {
-      const int R = id / D, cc = id - R * D;
+    for (int id = threadIdx.x; id < gn * DV; id += THREADS) {
+      const int R = id / DV, cc = id - R * DV;
       float M = -INFINITY;
 #pragma unroll
       for (int w = 0; w < 4; ++w) M = fmaxf(M, mml[(w * 16 + R) * 2]);
@@ -763,14 +768,14 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
       for (int w = 0; w < 4; ++w) {
         const float mw = mml[(w * 16 + R) * 2];
         const float f = mw == -INFINITY ? 0.f : exp2f(mw - M);
-        acc += mo[((size_t)w * 16 + R) * D + cc] * f;
+        acc += mo[((size_t)w * 16 + R) * DV + cc] * f;
         L += mml[(w * 16 + R) * 2 + 1] * f;
       }
       if (whole) {
         if (sinks && L > 0.f) L += exp2f(fmaf(sinks[kvh * G + g0 + R], LOG2E, -M));
-        out[tok * out_stride + (size_t)(kvh * G + g0 + R) * D + cc] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+        if (cc < out_head) out[tok * out_stride + (size_t)(kvh * G + g0 + R) * out_head + cc] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
       } else {
-        po[R * D + cc] = acc;
+        po[R * DV + cc] = acc;
         if (cc == 0) { pml[R * 2] = M; pml[R * 2 + 1] = L; }
       }
     }
@@ -785,7 +790,7 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
       }
       __syncthreads();
       if (s_flag == pieces - 1) {                              // the last piece to arrive: merge all, in piece order
-        const float* bo = part_o + unit * max_pieces * rows_per * D;
+        const float* bo = part_o + unit * max_pieces * rows_per * DV;
         const float* bml = part_ml + unit * max_pieces * rows_per * 2;
         // the pieces' (max, sum) first: few numbers, loaded side by side into shared memory
         float* sml = reinterpret_cast<float*>(smem_raw);       // [pieces][gn][2]
@@ -794,8 +799,8 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
           sml[id] = __ldcg(bml + (size_t)pc * rows_per * 2 + rem);
         }
         __syncthreads();
-        for (int id = threadIdx.x; id < gn * (D / 4); id += THREADS) {
-          const int R = id / (D / 4), c4 = id - R * (D / 4);
+        for (int id = threadIdx.x; id < gn * (DV / 4); id += THREADS) {
+          const int R = id / (DV / 4), c4 = id - R * (DV / 4);
           float M = -INFINITY;
           for (int pc = 0; pc < pieces; ++pc) M = fmaxf(M, sml[(pc * gn + R) * 2]);
           float L = 0.f;
@@ -804,7 +809,7 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
             float4 t[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-              t[j] = __ldcg(reinterpret_cast<const float4*>(bo + ((size_t)min(p0 + j, pieces - 1) * rows_per + R) * D) + c4);
+              t[j] = __ldcg(reinterpret_cast<const float4*>(bo + ((size_t)min(p0 + j, pieces - 1) * rows_per + R) * DV) + c4);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
               if (p0 + j >= pieces) break;
@@ -817,8 +822,8 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
           }
           if (sinks && L > 0.f) L += exp2f(fmaf(sinks[kvh * G + g0 + R], LOG2E, -M));
           const float inv = L > 0.f ? 1.0f / L : 0.f;
-          bf16* dst = out + tok * out_stride + (size_t)(kvh * G + g0 + R) * D + c4 * 4;
-          *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
+          bf16* dst = out + tok * out_stride + (size_t)(kvh * G + g0 + R) * out_head + c4 * 4;
+          if (c4 * 4 < out_head) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
         }
         if (threadIdx.x == 0) counters[unit] = 0;              // ready for the next launch
       }
@@ -853,7 +858,7 @@ NHV_API int NHV_FN(nhv_attn_mma_tile_d)() { return BN; }
 
 // The step's attention in bfloat16: prompt portions, then single tokens.
 // n_prefill_tokens / n_decode_seqs: how many of the step's tokens / requests are of each kind (0 skips that
-// launch).  Decoding needs scratch: scratch_o [n_seqs * head_blocks * max_pieces * rows * D] floats, scratch_ml
+// launch).  Decoding needs scratch: scratch_o [n_seqs * head_blocks * max_pieces * rows * DV] floats, scratch_ml
 // [... * rows * 2] floats and counters [n_seqs * head_blocks] ints that are zero (the kernel leaves them zero),
 // with head_blocks = nkv * ceil(group / 16), rows = min(group, 16), max_pieces >= ceil(longest context / 64) + 1.
 // decode_blocks: the grid of the decode kernel (a few blocks per SM).
@@ -862,7 +867,11 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
                             int n_seqs, int n_prefill_tokens, int n_prefill_seqs, int n_decode_seqs, int nq,
                             int nkv, int page_size, int n_pages, int window, int chunk, float scale, float* scratch_o,
                             float* scratch_ml, int* counters, int max_pieces, int decode_blocks,
-                            const FusedQK& fq, const float* sinks, const float* slopes, int keep_first, cudaStream_t stream) {
+                            const FusedQK& fq, const float* sinks, const float* slopes, int keep_first, int out_head,
+                            cudaStream_t stream) {
+  ATT_REQUIRE(out_head > 0 && out_head <= DV && out_head % 8 == 0,
+              "attention: an output head has %d elements, in steps of 8 up to %d", out_head, DV);
+  ATT_REQUIRE(!fq.qkv || (DV == D && out_head == D), "attention: the form that works from the projection has heads of one size");
   ATT_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention: kept first keys go with a window");
   ATT_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention: %d query heads do not divide into %d KV heads", nq, nkv);
   ATT_REQUIRE(page_size > 0 && n_pages > 0 && bt_stride > 0, "attention: bad page geometry");
@@ -903,12 +912,12 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
       if (wide)
         nhv_launch(attn_prefill_kernel<2>, grid, THREADS, prefill_smem_bytes<2>(), stream,
             (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv_pages, block_table, bt_stride, cu_q, kv_len,
-            n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first);
+            n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first, out_head);
     }
     if (!wide)
       nhv_launch(attn_prefill_kernel<1>, grid, THREADS, prefill_smem_bytes<1>(), stream,
           (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv_pages, block_table, bt_stride, cu_q, kv_len,
-          n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first);
+          n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first, out_head);
   }
   if (n_decode_seqs > 0) {
     ATT_REQUIRE(scratch_o && scratch_ml && counters && max_pieces > 0 && decode_blocks > 0,
@@ -925,7 +934,7 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
     decode_blocks = resident;
     nhv_launch(attn_decode_kernel, dim3(decode_blocks), THREADS, kDecodeSmemBytes, stream,
         (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv_pages, block_table, bt_stride, cu_q, kv_len,
-        scratch_o, scratch_ml, counters, n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, max_pieces, fq, sinks, slopes, keep_first);
+        scratch_o, scratch_ml, counters, n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, max_pieces, fq, sinks, slopes, keep_first, out_head);
   }
   const cudaError_t e = cudaPeekAtLastError();
   if (e != cudaSuccess) {
@@ -940,15 +949,16 @@ NHV_API int NHV_FN(nhv_attn_mma_d)(const void* q, int q_stride, void* out, int o
                                    int n_seqs, int n_prefill_tokens, int n_prefill_seqs, int n_decode_seqs, int nq,
                                    int nkv, int page_size, int n_pages, int window, int chunk, float scale, float* scratch_o,
                                    float* scratch_ml, int* counters, int max_pieces, int decode_blocks,
-                                   const float* sinks, const float* slopes, int keep_first, cudaStream_t stream) {
+                                   const float* sinks, const float* slopes, int keep_first, int out_head,
+                                   cudaStream_t stream) {
   FusedQK none = {};
   return attention_launch(q, q_stride, out, out_stride, kv_pages, block_table, bt_stride, cu_q, kv_len, n_seqs,
                           n_prefill_tokens, n_prefill_seqs, n_decode_seqs, nq, nkv, page_size, n_pages, window, chunk, scale,
-                          scratch_o, scratch_ml, counters, max_pieces, decode_blocks, none, sinks, slopes, keep_first, stream);
+                          scratch_o, scratch_ml, counters, max_pieces, decode_blocks, none, sinks, slopes, keep_first, out_head, stream);
 }
 
 // 1 if this head size has the form of the decode kernel that works from the projection's output.
-NHV_API int NHV_FN(nhv_attn_mma_can_fuse_d)() { return D % 32 == 0 ? 1 : 0; }
+NHV_API int NHV_FN(nhv_attn_mma_can_fuse_d)() { return D % 32 == 0 && DV == D ? 1 : 0; }
 
 // A step of single tokens only, straight from the projection's output qkv [tokens, (nq + 2 nkv) * D]: the kernel
 // norms and rotates the query and key heads itself and (store != 0) puts the new keys and values into the cache;
@@ -981,5 +991,5 @@ NHV_API int NHV_FN(nhv_attn_mma_decode_fused_d)(const void* qkv, int qkv_stride,
   fq.weight_offset = weight_offset;
   return attention_launch(qkv, qkv_stride, out, out_stride, kv_pages, block_table, bt_stride, cu_q, kv_len, n_seqs, 0, 0,
                           n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale, scratch_o, scratch_ml, counters, max_pieces,
-                          1, fq, nullptr, nullptr, 0, stream);
+                          1, fq, nullptr, nullptr, 0, D, stream);
 }

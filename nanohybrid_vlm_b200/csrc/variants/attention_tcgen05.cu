@@ -1,5 +1,7 @@
 // Attention of prompt portions over the paged cache on the 5th-generation tensor cores (tcgen05.mma, accumulators
-// in tensor memory, K and V brought by TMA), compiled per head size: -DNHV_ATTN_D=64|128|192|256.
+// in tensor memory, K and V brought by TMA), compiled per head size: -DNHV_ATTN_D=64|128|192|256, and per size of a
+// value head where that is smaller: -DNHV_ATTN_DV (a multiple of 64; page rows stay D wide, of a value row only the
+// first DV elements are read).
 //
 // softmax(q k^T * scale) v per query head, causal, optionally within a window, q of a portion's tokens against
 // all keys of the request that the cache holds (nanovllm/layers/attention.py:67-70 calls a library for this;
@@ -38,6 +40,9 @@
 #ifndef NHV_ATTN_D
 #error "compile with -DNHV_ATTN_D=<head size>"
 #endif
+#ifndef NHV_ATTN_DV
+#define NHV_ATTN_DV NHV_ATTN_D
+#endif
 #define NHV_CAT2(a, b) a##b
 #define NHV_CAT(a, b) NHV_CAT2(a, b)
 #define NHV_FN(name) NHV_CAT(name, NHV_ATTN_D)
@@ -45,20 +50,21 @@
 namespace {
 
 typedef __nv_bfloat16 bf16;
-constexpr int D = NHV_ATTN_D;
+constexpr int D = NHV_ATTN_D, DV = NHV_ATTN_DV;
 static_assert(D % 64 == 0 && D >= 64 && D <= 256, "head sizes 64, 128, 192 and 256");
+static_assert(DV % 64 == 0 && DV >= 64 && DV <= D, "value heads are a multiple of 64 up to the head size");
 constexpr int BM = 128;                      // rows of a block = lanes of tensor memory
 constexpr int BN = 64;                       // keys per tile
-constexpr int DB = D / 64;                   // 128-byte column blocks of a head
+constexpr int DB = D / 64, VB = DV / 64;     // 128-byte column blocks of a key head and of a value head
 constexpr int THREADS = 192;
 constexpr int Q_BYTES = DB * BM * 128;
-constexpr int T_BYTES = DB * BN * 128;       // one K tile or one V tile
+constexpr int T_BYTES = DB * BN * 128, V_BYTES = VB * BN * 128;     // one K tile, one V tile
 constexpr int STAGES = 2;
 constexpr int BAR_BYTES = 128;
-constexpr int SMEM_NEED = 1024 + Q_BYTES + 2 * STAGES * T_BYTES;    // barriers live in the first 128 bytes
+constexpr int SMEM_NEED = 1024 + Q_BYTES + STAGES * (T_BYTES + V_BYTES);    // barriers live in the first 128 bytes
 // at least 80 KB, so that an SM never holds more blocks than its tensor memory serves (two of 256 columns)
 constexpr int SMEM_BYTES = SMEM_NEED < 80 * 1024 ? 80 * 1024 : SMEM_NEED;
-constexpr uint32_t TMEM_COLS = (2 * BN + D) <= 256 ? 256 : 512;
+constexpr uint32_t TMEM_COLS = (2 * BN + DV) <= 256 ? 256 : 512;
 constexpr uint32_t S_COL = 0, O_COL = 2 * BN;
 constexpr float RESCALE_STEP = 8.0f;         // log2 units
 constexpr float LOG2E = 1.4426950408889634f;
@@ -164,12 +170,13 @@ struct alignas(64) Params {
   const float* sinks;     // per query head, or null: exp(sink) joins the softmax denominator (no key, no value, no scale)
   const float* slopes;    // per query head, or null: the score loses slopes[head] times the distance between query and key
   float inv_scale;        // 1 / scale: the distance term joins the raw score, which the exponent's multiply-add scales
+  int out_head;           // elements between two heads of the output, up to DV: that many are written
   int q_stride, out_stride, bt_stride, n_seqs, nq, nkv, page_size, n_pages, window, chunk, tokens_per_block;
   int keep_first;         // with a window: keys at positions below it stay visible (their tiles come first)
   float scale_log2;
 };
 
-__global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcgen05_kernel(const __grid_constant__ Params p) {
+__global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tcgen05_kernel(const __grid_constant__ Params p) {
   extern __shared__ __align__(128) unsigned char smem_raw[];
   // barriers in the first 128 bytes, the tiles from the next 1024-byte boundary on
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem_raw);
@@ -186,7 +193,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
   unsigned char* tiles = smem_raw + (((raw + BAR_BYTES + 1023u) & ~1023u) - raw);
   unsigned char* q_s = tiles;
   unsigned char* k_s = q_s + Q_BYTES;                  // [STAGES][T_BYTES]
-  unsigned char* v_s = k_s + STAGES * T_BYTES;         // [STAGES][T_BYTES]
+  unsigned char* v_s = k_s + STAGES * T_BYTES;         // [STAGES][V_BYTES]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -273,9 +280,9 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
 #pragma unroll
         for (int b = 0; b < DB; ++b) tma_load_2d(k_s + st * T_BYTES + b * (BN * 128), &p.kv_map, b * 64, row_k, &k_full[st]);
         if (j >= STAGES && !mbar_wait(&v_empty[st], (uint32_t)((j >> 1) - 1) & 1, 2)) { *s_abort = 1; issued = j; break; }
-        mbar_expect_tx(&v_full[st], T_BYTES);
+        mbar_expect_tx(&v_full[st], V_BYTES);
 #pragma unroll
-        for (int b = 0; b < DB; ++b) tma_load_2d(v_s + st * T_BYTES + b * (BN * 128), &p.kv_map, b * 64, row_v, &v_full[st]);
+        for (int b = 0; b < VB; ++b) tma_load_2d(v_s + st * V_BYTES + b * (BN * 128), &p.kv_map, b * 64, row_v, &v_full[st]);
         issued = j + 1;
         page = page_next;
       }
@@ -292,7 +299,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0 && n_tiles > 0) {
       const uint32_t idesc_s = instr_desc(BM, BN, false);
-      const uint32_t idesc_o = instr_desc(BM, D, true);
+      const uint32_t idesc_o = instr_desc(BM, DV, true);
       // descriptors are made once: a later K slice, column block or stage only moves the start address, which
       // sits in the low bits in units of 16 bytes
       const uint64_t q_desc = smem_desc(smem_u32(q_s), 16, 1024);
@@ -321,7 +328,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
         ok = mbar_wait(p_ready, (uint32_t)j & 1, 5) && mbar_wait(&v_full[st], (uint32_t)(j >> 1) & 1, 6);
         if (!ok) break;
         tc_fence_after();
-        const uint64_t vd = v_desc + (uint64_t)(st * (T_BYTES >> 4));
+        const uint64_t vd = v_desc + (uint64_t)(st * (V_BYTES >> 4));
         const uint32_t p_addr = tmem_base + S_COL + (uint32_t)((j & 1) * BN);    // P lies over the first half of this tile's S
 #pragma unroll
         for (int kk = 0; kk < BN / 16; ++kk)                                       // 8 columns of P and 16 rows of V per 16 keys
@@ -411,7 +418,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
         tc_fence_after();
         if (__any_sync(0xffffffffu, grow)) {
 #pragma unroll 1
-          for (int c0 = 0; c0 < D; c0 += 32) {
+          for (int c0 = 0; c0 < DV; c0 += 32) {
             uint32_t o[32];
             tmem_ld32_nowait(o, lane_addr + O_COL + c0);
             tmem_ld_wait();
@@ -431,9 +438,9 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
         ok = mbar_wait(&v_full[j & 1], (uint32_t)(j >> 1) & 1, 10);
         if (!ok) break;
         const int first_bad = total - key_base;                  // 1..63
-        for (int id = threadIdx.x - 64; id < (BN - first_bad) * DB * 8; id += 128) {
-          const int row = first_bad + id / (DB * 8), rem = id % (DB * 8);
-          *reinterpret_cast<uint4*>(v_s + (j & 1) * T_BYTES + (rem >> 3) * (BN * 128) + row * 128 + ((rem & 7) << 4)) =
+        for (int id = threadIdx.x - 64; id < (BN - first_bad) * VB * 8; id += 128) {
+          const int row = first_bad + id / (VB * 8), rem = id % (VB * 8);
+          *reinterpret_cast<uint4*>(v_s + (j & 1) * V_BYTES + (rem >> 3) * (BN * 128) + row * 128 + ((rem & 7) << 4)) =
               make_uint4(0, 0, 0, 0);
         }
         fence_async_smem();
@@ -447,9 +454,9 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
       // the sink: one more term of the sum, in the units of the running reference (an overflow to inf gives inv = 0)
       if (p.sinks && valid && l > 0.f) l += exp2f(fmaf(p.sinks[kvh * G + g], LOG2E, -m_run));
       const float inv = l > 0.f ? 1.0f / l : 0.f;
-      bf16* dst = p.out + (size_t)(q_row0 + t0 + tq) * p.out_stride + (size_t)(kvh * G + g) * D;
+      bf16* dst = p.out + (size_t)(q_row0 + t0 + tq) * p.out_stride + (size_t)(kvh * G + g) * p.out_head;
 #pragma unroll 1
-      for (int c0 = 0; c0 < D; c0 += 32) {
+      for (int c0 = 0; c0 < DV; c0 += 32) {
         uint32_t o[32];
         tmem_ld32_nowait(o, lane_addr + O_COL + c0);
         tmem_ld_wait();
@@ -461,7 +468,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + D) <= 256 ? 2 : 1) attn_tcg
             w.y = pack_bf16(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
             w.z = pack_bf16(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
             w.w = pack_bf16(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
-            *reinterpret_cast<uint4*>(dst + c0 + i) = w;
+            if (c0 + i < p.out_head) *reinterpret_cast<uint4*>(dst + c0 + i) = w;
           }
         }
       }
@@ -526,7 +533,9 @@ NHV_API int NHV_FN(nhv_attn_tcgen05_d)(const void* q, int q_stride, void* out, i
                                        const int* block_table, int bt_stride, const int* cu_q, const int* kv_len,
                                        int n_seqs, int n_prefill_tokens, int n_prefill_seqs, int nq, int nkv,
                                        int page_size, int n_pages, int window, int chunk, float scale, const float* sinks,
-                                       const float* slopes, int keep_first, cudaStream_t stream) {
+                                       const float* slopes, int keep_first, int out_head, cudaStream_t stream) {
+  ATT_REQUIRE(out_head > 0 && out_head <= DV && out_head % 8 == 0,
+              "attention (tcgen05): an output head has %d elements, in steps of 8 up to %d", out_head, DV);
   ATT_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention: kept first keys go with a window");
   ATT_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention: %d query heads do not divide into %d KV heads", nq, nkv);
   const int G = nq / nkv;
@@ -561,6 +570,7 @@ NHV_API int NHV_FN(nhv_attn_tcgen05_d)(const void* q, int q_stride, void* out, i
   p.slopes = slopes;
   p.inv_scale = 1.0f / scale;
   ATT_REQUIRE(slopes == nullptr || scale > 0.f, "attention (tcgen05): a distance term needs a positive scale");
+  p.out_head = out_head;
   p.q_stride = q_stride;
   p.out_stride = out_stride;
   p.bt_stride = bt_stride;

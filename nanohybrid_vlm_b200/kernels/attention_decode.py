@@ -24,14 +24,17 @@ def supports(head_dim: int, nq: int, nkv: int, page_size: int, n_seqs: int = 1) 
             and page_size % TILE == 0 and n_seqs <= MAX_SEQS)
 
 
-def get(head_dim: int):
-    """(launch function, blocks of a launch) for this head size.  The kernel's error word is registered with
+def get(head_dim: int, v_dim: int | None = None):
+    """(launch function, blocks of a launch) for this head size (``v_dim``: the size that the value heads are compiled
+    for, where it is smaller).  The kernel's error word is registered with
     the step's health word (``ops.register_wait_error_source``)."""
-    if head_dim not in _libs:
+    v_dim = v_dim or head_dim
+    key = head_dim if v_dim == head_dim else (head_dim, v_dim)
+    if key not in _libs:
         from ..csrc.build import ensure_variant
-        lib = ctypes.CDLL(ensure_variant("attention_decode.cu", {"NHV_ATTN_D": head_dim}))
+        lib = ctypes.CDLL(ensure_variant("attention_decode.cu", {"NHV_ATTN_D": head_dim, **({} if v_dim == head_dim else {"NHV_ATTN_DV": v_dim})}))
         fn = getattr(lib, f"nhv_attn_decode_d{head_dim}")
-        fn.argtypes = [P, I, P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, F, P, P, P, P, P, P, P, P, I, I, I, F, F, P, I, P]
+        fn.argtypes = [P, I, P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, F, P, P, P, P, P, P, P, P, I, I, I, F, F, P, I, I, P]
         fn.restype = c_int
         err = getattr(lib, f"nhv_attn_decode_last_error_d{head_dim}")
         err.restype = ctypes.c_char_p
@@ -42,11 +45,11 @@ def get(head_dim: int):
         blocks = getattr(lib, f"nhv_attn_decode_blocks_d{head_dim}")
         blocks.restype = c_int
         from . import ops
-        ops.register_wait_error_source(f"attention_decode (head size {head_dim})", address, take)
+        ops.register_wait_error_source(f"attention_decode (head size {head_dim}{'' if v_dim == head_dim else f', values {v_dim}'})", address, take)
 
         def launch(*args, _fn=fn, _err=err):
             if _fn(*args) != 0:
                 raise KernelError(_err().decode(errors="replace"))
 
-        _libs[head_dim] = (launch, blocks())
-    return _libs[head_dim]
+        _libs[key] = (launch, blocks())
+    return _libs[key]

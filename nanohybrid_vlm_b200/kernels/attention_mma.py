@@ -24,14 +24,23 @@ def supports(head_dim: int, nq: int, nkv: int, n_seqs: int = 1) -> bool:
             and n_seqs <= MAX_SEQS)
 
 
-def get(head_dim: int):
+def value_size(head_dim: int, v_head: int) -> int:
+    """The size that value heads of ``v_head`` elements are compiled for beside keys of ``head_dim``: the next multiple of
+    64 where the key heads are one (every kernel takes it), else of 16."""
+    step = 64 if head_dim % 64 == 0 else 16
+    return min(head_dim, -(-v_head // step) * step)
+
+
+def get(head_dim: int, v_dim: int | None = None):
     """(launch function, keys per tile, launch function of the decode form that works from the projection's
-    output, or None) for this head size."""
-    if head_dim not in _libs:
+    output, or None) for this head size (``v_dim``: the size that the value heads are compiled for, where it is smaller)."""
+    v_dim = v_dim or head_dim
+    key = head_dim if v_dim == head_dim else (head_dim, v_dim)
+    if key not in _libs:
         from ..csrc.build import ensure_variant
-        lib = ctypes.CDLL(ensure_variant("attention_mma.cu", {"NHV_ATTN_D": head_dim}))
+        lib = ctypes.CDLL(ensure_variant("attention_mma.cu", {"NHV_ATTN_D": head_dim, **({} if v_dim == head_dim else {"NHV_ATTN_DV": v_dim})}))
         fn = getattr(lib, f"nhv_attn_mma_d{head_dim}")
-        fn.argtypes = [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, I, P, P, I, P]
+        fn.argtypes = [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, I, P, P, I, I, P]
         fn.restype = c_int
         err = getattr(lib, f"nhv_attn_mma_last_error_d{head_dim}")
         err.restype = ctypes.c_char_p
@@ -52,5 +61,5 @@ def get(head_dim: int):
             if _fn(*args) != 0:
                 raise KernelError(_err().decode(errors="replace"))
 
-        _libs[head_dim] = (launch, split(), launch_fused if can_fuse() else None)
-    return _libs[head_dim]
+        _libs[key] = (launch, split(), launch_fused if can_fuse() else None)
+    return _libs[key]

@@ -22,14 +22,17 @@ def supports(head_dim: int, nq: int, nkv: int, page_size: int) -> bool:
             and page_size % TILE == 0)
 
 
-def get(head_dim: int):
-    """(launch function, function that reads and clears the error word) for this head size.  The error word is
+def get(head_dim: int, v_dim: int | None = None):
+    """(launch function, function that reads and clears the error word) for this head size (``v_dim``: the size that the
+    value heads are compiled for, where it is smaller).  Launches end with the elements of an output head and the stream.  The error word is
     also registered with the step's health word (``ops.register_wait_error_source``)."""
-    if head_dim not in _libs:
+    v_dim = v_dim or head_dim
+    key = head_dim if v_dim == head_dim else (head_dim, v_dim)
+    if key not in _libs:
         from ..csrc.build import ensure_variant
-        lib = ctypes.CDLL(ensure_variant("attention_tcgen05.cu", {"NHV_ATTN_D": head_dim}))
+        lib = ctypes.CDLL(ensure_variant("attention_tcgen05.cu", {"NHV_ATTN_D": head_dim, **({} if v_dim == head_dim else {"NHV_ATTN_DV": v_dim})}))
         fn = getattr(lib, f"nhv_attn_tcgen05_d{head_dim}")
-        fn.argtypes = [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, F, P, P, I, P]
+        fn.argtypes = [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, F, P, P, I, I, P]
         fn.restype = c_int
         err = getattr(lib, f"nhv_attn_tcgen05_last_error_d{head_dim}")
         err.restype = ctypes.c_char_p
@@ -38,11 +41,11 @@ def get(head_dim: int):
         address = getattr(lib, f"nhv_attn_tcgen05_error_word_d{head_dim}")
         address.restype, address.argtypes = c_void_p, []
         from . import ops
-        ops.register_wait_error_source(f"attention_tcgen05 (head size {head_dim})", address, word)
+        ops.register_wait_error_source(f"attention_tcgen05 (head size {head_dim}{'' if v_dim == head_dim else f', values {v_dim}'})", address, word)
 
         def launch(*args, _fn=fn, _err=err):
             if _fn(*args) != 0:
                 raise KernelError(_err().decode(errors="replace"))
 
-        _libs[head_dim] = (launch, word)
-    return _libs[head_dim]
+        _libs[key] = (launch, word)
+    return _libs[key]

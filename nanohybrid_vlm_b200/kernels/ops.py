@@ -895,13 +895,14 @@ SINK_ATTENTION_ON_TENSOR_CORES = True     # tests switch it off to compare with 
 def attention_sink(out, q, kv_pages, tables, batch, nq: int, nkv: int, dk: int, dv: int, scale: float, sinks=None,
                    window: int = 0, chunk: int = 0, slopes=None, keep_first: int = 0) -> None:
     """Attention of the step's tokens over the cache for layers with a sink and / or value heads of another size
-    than their key heads: picks the kernel for the dtype and sizes.  bfloat16 with key and value heads of one size
-    (in steps of 16) runs on the tensor cores like ``attention``; float32 and unequal head sizes on the CUDA cores."""
-    if (SINK_ATTENTION_ON_TENSOR_CORES and q.dtype == torch.bfloat16 and dk == dv and kv_pages.shape[-1] == dk
+    than their key heads: picks the kernel for the dtype and sizes.  bfloat16 with page rows and key heads of one size
+    (in steps of 16) and value heads of at most that size (in steps of 8) runs on the tensor cores like ``attention``;
+    float32 and other head sizes on the CUDA cores."""
+    if (SINK_ATTENTION_ON_TENSOR_CORES and q.dtype == torch.bfloat16 and dv <= dk and dv % 8 == 0 and kv_pages.shape[-1] == dk
             and kv_pages.shape[1] == 2 and attention_mma.supports(dk, nq, nkv, batch.n_seqs)):
         attention_tensor_core(out, q, kv_pages, tables.block_tables, batch.cu_q, batch.kv_len, batch.n_seqs,
                               batch.n_prefill_tokens, batch.n_prefill_seqs, batch.n_decode_seqs, batch.max_kv_len,
-                              nq, nkv, dk, scale, window, sinks, chunk, slopes, keep_first)
+                              nq, nkv, dk, scale, window, sinks, chunk, slopes, keep_first, dv)
         return
     attention_sink_simt(out, q, kv_pages, tables.block_tables, batch.cu_q, batch.kv_len, batch.n_seqs, batch.n_tokens,
                         nq, nkv, dk, dv, scale, sinks, window, chunk, slopes, keep_first)
@@ -1014,8 +1015,9 @@ def _attention_decode_tma(out, q, qkv, kv_pages, block_table, batch_cu_q, batch_
                           head_dim: int, scale: float, window: int, q_weight=None, k_weight=None, cos_sin=None,
                           positions=None, slot_mapping=None, rotary_dim: int = 0, eps: float = 0.0,
                           weight_offset: float = 0.0, store: bool = False, sinks=None, chunk: int = 0,
-                          keep_first: int = 0) -> None:
-    launch, blocks = attention_decode.get(head_dim)
+                          keep_first: int = 0, v_head: int | None = None) -> None:
+    v_head = v_head or head_dim
+    launch, blocks = attention_decode.get(head_dim, attention_mma.value_size(head_dim, v_head))
     n_pages, two, h, page_size, d = kv_pages.shape
     group = nq // nkv
     head_blocks = nkv * -(-group // 16)
@@ -1027,7 +1029,7 @@ def _attention_decode_tma(out, q, qkv, kv_pages, block_table, batch_cu_q, batch_
            batch_kv_len.data_ptr(), n_seqs, nq, nkv, page_size, n_pages, int(window), int(chunk), float(scale), part_o.data_ptr(),
            part_ml.data_ptr(), counters.data_ptr(), _ptr(q_weight), _ptr(k_weight), _ptr(cos_sin), _ptr(positions),
            _ptr(slot_mapping), int(rotary_dim), 0 if cos_sin is None else cos_sin.shape[0], 1 if store else 0, float(eps),
-           float(weight_offset), _ptr(sinks), int(keep_first), stream_ptr())
+           float(weight_offset), _ptr(sinks), int(keep_first), v_head, stream_ptr())
 
 
 def attention_decode_fused(out, qkv, kv_pages, tables, batch, nq: int, nkv: int, head_dim: int, scale: float,
@@ -1087,7 +1089,8 @@ def attention_tcgen05_error(head_dim: int) -> int:
 
 def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: int, n_prefill_tokens: int,
                           n_prefill_seqs: int, n_decode_seqs: int, max_kv_len: int, nq: int, nkv: int, head_dim: int,
-                          scale: float, window: int = 0, sinks=None, chunk: int = 0, slopes=None, keep_first: int = 0) -> None:
+                          scale: float, window: int = 0, sinks=None, chunk: int = 0, slopes=None, keep_first: int = 0,
+                          v_head: int | None = None) -> None:
     """bfloat16 attention on the tensor cores.  Prompt portions go to the tcgen05 kernel, requests with
     one new token to the kernel that streams the cache with TMA, each where its shape is supported; what
     neither takes runs in the mma.sync kernel, whose single-token path shares a request's tiles between
@@ -1096,7 +1099,9 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
     ``slopes`` [nq] float32: head h's score loses slopes[h] times the distance between query and key; the tcgen05 and
     the mma.sync kernels take them, the TMA kernel for single tokens does not, so those run in the mma.sync kernel.
     ``keep_first`` > 0 (with a window): the keys at positions below it stay visible; in every kernel their tiles come
-    before the window's."""
+    before the window's.
+    ``v_head`` (in steps of 8, up to ``head_dim``): the elements of a value head, where they are fewer: the leading ones
+    of a page's value row; out is then [T, nq * v_head]."""
     _need_cuda(out, q, kv_pages, block_table, cu_q, kv_len, sinks, slopes)
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == nq and sinks.is_contiguous())
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == nq and slopes.is_contiguous())
@@ -1105,16 +1110,18 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
     n_pages, two, h, page_size, d = kv_pages.shape
     assert two == 2 and h == nkv and d == head_dim
     assert block_table.dtype == torch.int32 and block_table.stride(-1) == 1
-    launch, tile = attention_mma.get(head_dim)[:2]
+    v_head = v_head or head_dim
+    v_dim = attention_mma.value_size(head_dim, v_head)
+    launch, tile = attention_mma.get(head_dim, v_dim)[:2]
     if (n_prefill_tokens > 0 and USE_TCGEN05_ATTENTION and (slopes is None or scale > 0)
             and attention_tcgen05.supports(head_dim, nq, nkv, page_size)):
         # prompt portions on the 5th-generation tensor cores; single tokens stay with the split kernel below
         library.LAUNCHES += 1
-        attention_tcgen05.get(head_dim)[0](
+        attention_tcgen05.get(head_dim, v_dim)[0](
             q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), kv_pages.data_ptr(), block_table.data_ptr(),
             block_table.stride(0), cu_q.data_ptr(), kv_len.data_ptr(), n_seqs, n_prefill_tokens, n_prefill_seqs,
             nq, nkv, page_size, n_pages, int(window), int(chunk), float(scale), _ptr(sinks), _ptr(slopes), int(keep_first),
-            stream_ptr())
+            v_head, stream_ptr())
         if n_decode_seqs == 0:
             return
         n_prefill_tokens = n_prefill_seqs = 0
@@ -1123,7 +1130,7 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
         # single tokens: the kernel that streams the cache with TMA; what is left for the launch below are the
         # prompt portions (if the tcgen05 kernel did not take them)
         _attention_decode_tma(out, q, None, kv_pages, block_table, cu_q, kv_len, n_seqs, nq, nkv, head_dim, scale, window,
-                              sinks=sinks, chunk=chunk, keep_first=keep_first)
+                              sinks=sinks, chunk=chunk, keep_first=keep_first, v_head=v_head)
         if n_prefill_tokens == 0:
             return
         n_decode_seqs = 0
@@ -1143,7 +1150,7 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
     launch(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), kv_pages.data_ptr(), block_table.data_ptr(),
            block_table.stride(0), cu_q.data_ptr(), kv_len.data_ptr(), n_seqs, n_prefill_tokens, n_prefill_seqs,
            n_decode_seqs, nq, nkv, page_size, n_pages, int(window), int(chunk), float(scale), _ptr(scratch_o), _ptr(scratch_ml),
-           _ptr(counters), max_pieces, blocks, _ptr(sinks), _ptr(slopes), int(keep_first), stream_ptr())
+           _ptr(counters), max_pieces, blocks, _ptr(sinks), _ptr(slopes), int(keep_first), v_head, stream_ptr())
 
 
 _sm_counts: dict = {}

@@ -133,13 +133,16 @@ class LatentAttention(Mixer):
         T, H, D = q.shape[0], self.H, self.D
         qp, pages, tables = ops.latent_expand(cache.pages, cache.tables, batch, q, q_lat, self.ukv, H, self.dn, self.dr,
                                               self.dv, self.rank, D, self.window or 0)
-        padded = self.new(T, H * D)
+        # value heads in steps of 8 leave the kernels as they are; others in padded heads
+        own = self.dv % 8 == 0
+        padded = self.new(T, H * (self.dv if own else D))
         ops.attention_tensor_core(padded, qp, pages, tables, batch.cu_q, batch.kv_len, batch.n_seqs,
                                   batch.n_prefill_tokens, batch.n_prefill_seqs, batch.n_decode_seqs, batch.max_kv_len, H, H,
-                                  D, self.scale, self.window or 0, self.w_sink if self.has_sink else None)
-        o = padded if D == self.dv and not self.gate else self.new(T, H * self.dv)
+                                  D, self.scale, self.window or 0, self.w_sink if self.has_sink else None,
+                                  v_head=self.dv if own else D)
+        o = padded if own and not self.gate else self.new(T, H * self.dv)
         if self.gate:
-            ops.sigmoid_mul_heads(o, padded, gate, self.dv, x_head=D)
+            ops.sigmoid_mul_heads(o, padded, gate, self.dv, x_head=None if own else D)
         elif o is not padded:
             o.view(T, H, self.dv).copy_(padded.view(T, H, D)[:, :, :self.dv])
         y = self.new(T, self.env.hidden_size)
