@@ -7,6 +7,7 @@
     python bench.py --designs nomudra        Nomudra beside a Muvonex of equal active size, the same way
     python bench.py --designs ginodra        Ginodra beside a Muvonex of equal size, the same way
     python bench.py --designs beputar        Beputar beside a Nomudra of the same width and expert sizes, the same way
+    python bench.py --designs vozorax        Vozorax beside a Ginodra of equal active size and a Nomudra, the same way
 
 The default run has the layer sizes of the Qwen3-8B-shaped configuration (36 layers, width 4096,
 32/8 heads of 128, feed-forward 12288, vocabulary 151936), bfloat16, random weights, batch 8,
@@ -724,6 +725,22 @@ def beputar_config(width: int, heads: int, ff: int, layers: int) -> dict:
                 layers=[kinds[i % 4] for i in range(layers)], dtype="bfloat16")
 
 
+def vozorax_config(width: int, heads: int, ff: int, layers: int) -> dict:
+    """In turn: attention over latents in a window of 1,024 (heads of 128 + 64 rotated, a latent of 512, queries through a
+    latent of 3/8 of the width) and attention in a window of 1,024 with sinks and mixed values (a quarter as many key
+    heads); four copies of the residual stream.  The first layer of every four has the dense feed-forward ``ff``; the
+    others a mixture of 16 experts of two matrices of which a token uses 4, and a shared expert: they hold what the
+    dense one's three matrices hold (4 * 3/11 + 9/22 of ``ff``, times two matrices)."""
+    moe = dict(kind="moe", router=dict(experts=16, top=4), expert=dict(ff=ff * 3 // 11), shared=dict(ff=ff * 9 // 22 // 8 * 8))
+    latent = dict(type="latent_attention", mixer=dict(
+        heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=width * 3 // 8, kv_rank=512, scale=192 ** -0.5,
+        rot=dict(base=10000.0, dims=64), mask=dict(size=1024)))
+    window = dict(type="attention", mixer=dict(heads=heads, kv_heads=max(heads // 4, 1), dim=128, vdim=64, scale=128 ** -0.5,
+                                               mask=dict(size=1024), v_mix=True))
+    return dict(architecture="Vozorax", vocab=DESIGN_VOCAB, width=width, streams=4, norm=dict(eps=1e-6), dtype="bfloat16",
+                layers=[dict((latent, window)[i % 2], mlp=dict(kind="dense", ff=ff) if i % 4 == 0 else moe) for i in range(layers)])
+
+
 def qwen3_config_of_equal_size(width: int, heads: int, layers: int, layer_weights: float) -> dict:
     """A Qwen3 of this width whose layers hold as many weights as ``layer_weights`` (the feed-forward takes up the
     difference, rounded to 256)."""
@@ -738,7 +755,8 @@ def bench_designs(args) -> dict:
     """Prefill and decode throughput of Muvonex beside a Qwen3 of equal size (``--designs``), or of Nomudra beside a
     Muvonex whose layers hold as many weights as a Nomudra token uses (``--designs nomudra``), or of Ginodra beside a
     Muvonex of equal size (``--designs ginodra``), or of Beputar beside a Nomudra of the same width and expert sizes
-    (``--designs beputar``), and the time of each kind
+    (``--designs beputar``), or of Vozorax beside a Ginodra whose layers hold as many weights as a Vozorax token uses and
+    beside a Nomudra of the same width (``--designs vozorax``), and the time of each kind
     of kernel in a prefill step (CUDA events around every launch of an eager run) with its share of the measured
     roofline."""
     import torch
@@ -761,7 +779,8 @@ def bench_designs(args) -> dict:
              "latent_rope_store": "rope_store", "linear_heads": "gemm_heads", "attention_sink_simt": "attention",
              "latent_attention": "attention", "latent_expand": "attention", "general_delta": "delta_rule", "sigmoid_mul_heads": "act_mul",
              "relu_squared": "act_mul", "scale_softcap": "act_mul", "gelu_tanh": "act_mul", "postnorm_stream": "norm",
-             "stream_round": "norm", "token_shift_mix": "token_shift", "decay_scan": "decay_scan", "decay_lowrank": "decay_prep"}
+             "stream_round": "norm", "token_shift_mix": "token_shift", "decay_scan": "decay_scan", "decay_lowrank": "decay_prep",
+             "streams_rmsnorm": "norm", "row_norm_store": "rope_store"}
     kinds = {k: v for k, v in kinds.items() if hasattr(ops, k)}
     stock = {name: getattr(ops, name) for name in kinds}
     gen = torch.Generator().manual_seed(SEED)
@@ -795,7 +814,8 @@ def bench_designs(args) -> dict:
         expert_weights = sum(e * r * c for e, r, c in stacks)
         tops = [dict(lay.ffn.spec.items) for lay in runner.model.spec.layers if "ffn" in dict(lay.parts)
                 and lay.ffn.spec.kind == "routed_moe"]
-        used = sum(3 * t["top"] * t["intermediate_size"] * cfg.get("width", 0) for t in tops)
+        matrices = [2 if t.get("unit") == "relu2" else 3 for t in tops]        # of one expert
+        used = sum(n * t["top"] * t["intermediate_size"] * cfg.get("width", 0) for n, t in zip(matrices, tops))
         prompt = torch.randint(0, vocab, (T,), generator=gen).tolist()
         events, depth = [], [0]
 
@@ -879,7 +899,7 @@ def bench_designs(args) -> dict:
             ms = e0.elapsed_time(e1) / steps
             item = 2
             # of a stack of E experts a step reads those that some token chose: at most batch * top of them
-            hit = sum(min(e, batch * t["top"]) * r * c for (e, r, c), t in zip(stacks, [t for t in tops for _ in range(3)]))
+            hit = sum(min(e, batch * t["top"]) * r * c for (e, r, c), t in zip(stacks, [t for n, t in zip(matrices, tops) for _ in range(n)]))
             read = (weights + hit) * item + sum(runner.layout.page_bytes(page, torch.bfloat16)) * batch * (ctx // page) \
                 + runner.layout.state_bytes_per_slot(torch.bfloat16) * batch * 2
             out[f"decode_b{batch}"] = {"ms_per_step": round(ms, 3), "tok_s": round(batch / ms * 1e3),
@@ -930,6 +950,15 @@ def bench_designs(args) -> dict:
             ff = max(256, int(round((sz["ff"] + (per_layer - m0 / layers) / (3 * sz["width"])) / 256)) * 256)
             results[name] = {"ginodra": g, "muvonex": run_one(muvonex_config(sz["width"], sz["heads"], ff, layers), DESIGN_VOCAB)}
             continue
+        if args.designs == "vozorax":
+            v = run_one(vozorax_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB)
+            # a Ginodra whose dense feed-forward makes up for the difference in the mixers' weights
+            per_layer = (v["weights_a_token_uses_m"] * 1e6 - 2 * DESIGN_VOCAB * sz["width"]) / layers      # a head of its own
+            g0 = run_one_weights(ginodra_config(sz["width"], sz["heads"], sz["ff"], layers))
+            ff = max(256, int(round((sz["ff"] + (per_layer - g0 / layers) / (3 * sz["width"])) / 256)) * 256)
+            results[name] = {"vozorax": v, "ginodra": run_one(ginodra_config(sz["width"], sz["heads"], ff, layers), DESIGN_VOCAB),
+                             "nomudra": run_one(nomudra_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB)}
+            continue
         if args.designs == "beputar":
             # the same width, heads, expert count and expert sizes: both report the weights that a token uses
             results[name] = {"beputar": run_one(beputar_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB),
@@ -966,7 +995,7 @@ def main() -> int:
     ap.add_argument("--requests", type=int, default=0, help="fewer requests than the workload names (trying it out)")
     ap.add_argument("--breakdown", action="store_true",
                     help="time by kind of kernel in an eager run with --layers layers (default 2); prints one JSON line")
-    ap.add_argument("--designs", nargs="?", const="muvonex", default=None, choices=["muvonex", "nomudra", "ginodra", "beputar"],
+    ap.add_argument("--designs", nargs="?", const="muvonex", default=None, choices=["muvonex", "nomudra", "ginodra", "beputar", "vozorax"],
                     help="two designs side by side, prefill and decode throughput at a few layer sizes, one JSON line: "
                          "Muvonex beside a Qwen3 of equal size (the default), or Nomudra beside a Muvonex of equal active size")
     ap.add_argument("--design-size", default="all", choices=["all", *DESIGN_SIZES], help="one size of --designs")

@@ -161,7 +161,7 @@ def test_latent_attention_in_a_window(ops, dtype, m, page, expand, monkeypatch):
         rope_layout="interleaved", position=part("rope_banded", theta=m["rot"]["base"], rotary_dim=m["rot"]["dims"])),
         W, dtype, 11)
     x = [torch.randn(n, W, generator=torch.Generator().manual_seed(n)).to(dtype) for n in LENGTHS]
-    rig = Rig([mixer.cache_need()], page_size=page, num_pages=-(-300 // page), dtype=dtype)
+    rig = Rig([mixer.cache_need()], page_size=page, num_pages=-(-300 // page) + 4, dtype=dtype)
 
     def step(b, rows):
         return mixer.forward(dev(torch.cat([x[r][s:s + n] for r, s, n in rows])), b, rig.view(0, b))
@@ -241,7 +241,7 @@ def test_attention_with_whole_norms_sinks_and_mixed_values(ops, dtype, m, page):
                                    qk_norm_weight=True, qk_norm_scope="projection", sink=True, window=size, value_mix=vm),
                       W, dtype, 20 + i, scale={"sink": 2.0}) for i, vm in enumerate(("source", "mixed", None))]
     x = [[torch.randn(n, W, generator=torch.Generator().manual_seed(10 * n + i)).to(dtype) for n in LENGTHS] for i in range(3)]
-    rig = Rig([p.cache_need() for p, _ in made], page_size=page, num_pages=-(-300 // page), dtype=dtype)
+    rig = Rig([p.cache_need() for p, _ in made], page_size=page, num_pages=-(-300 // page) + 4, dtype=dtype)
 
     def step(b, rows):
         return torch.cat([p.forward(dev(torch.cat([x[i][r][s:s + n] for r, s, n in rows])), b, rig.view(i, b))
