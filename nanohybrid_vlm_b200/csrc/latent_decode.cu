@@ -270,28 +270,64 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(
 }
 
 // out[tok, h, :] = sum over splits of part_o * 2^(m - M) / (sum of l * 2^(m - M) + 2^(sink - M)); one block per (tok, h).
-__global__ void latent_decode_merge_kernel(bf16* __restrict__ out, int out_stride, const float* __restrict__ part_o,
-                                           const float* __restrict__ part_ml, const float* __restrict__ sinks, int H,
-                                           int rank, int n_splits) {
+// The splits' factors (at most LD_MAX_SPLITS) are made once by the first warp; a thread then sums four columns, its loads
+// of several splits on their way at a time.
+constexpr int LD_MAX_SPLITS = 64;
+
+__global__ void __launch_bounds__(128) latent_decode_merge_kernel(bf16* __restrict__ out, int out_stride,
+                                           const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                           const float* __restrict__ sinks, int H, int rank, int n_splits) {
+  __shared__ float factor[LD_MAX_SPLITS];
+  __shared__ float s_inv;
   pdl_prologue();
   const int tok = blockIdx.x / H, h = blockIdx.x % H;
   const size_t base = ((size_t)tok * H + h) * n_splits;
-  float M = sinks ? sinks[h] * LD_LOG2E : -INFINITY;
-  for (int i = 0; i < n_splits; ++i)
-    if (part_ml[(base + i) * 2 + 1] > 0.f) M = fmaxf(M, part_ml[(base + i) * 2]);
-  float L = sinks ? exp2f(sinks[h] * LD_LOG2E - M) : 0.f;
-  for (int i = 0; i < n_splits; ++i) {
-    const float l = part_ml[(base + i) * 2 + 1];
-    if (l > 0.f) L += l * exp2f(part_ml[(base + i) * 2] - M);
-  }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
-  for (int c = threadIdx.x; c < rank; c += blockDim.x) {
-    float acc = 0.f;
-    for (int i = 0; i < n_splits; ++i) {
-      const float l = part_ml[(base + i) * 2 + 1];
-      if (l > 0.f) acc = fmaf(part_o[(base + i) * rank + c], exp2f(part_ml[(base + i) * 2] - M), acc);
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    float m[LD_MAX_SPLITS / 32], l[LD_MAX_SPLITS / 32];
+    float M = sinks ? sinks[h] * LD_LOG2E : -INFINITY;
+#pragma unroll
+    for (int k = 0; k < LD_MAX_SPLITS / 32; ++k) {
+      const int i = lane + 32 * k;
+      const float2 ml = i < n_splits ? *reinterpret_cast<const float2*>(part_ml + (base + i) * 2) : make_float2(-INFINITY, 0.f);
+      m[k] = ml.x;
+      l[k] = ml.y;
+      if (ml.y > 0.f) M = fmaxf(M, ml.x);
     }
-    out[(size_t)tok * out_stride + (size_t)h * rank + c] = __float2bfloat16_rn(acc * inv);
+    M = warp_max(M);
+    float L = 0.f;
+#pragma unroll
+    for (int k = 0; k < LD_MAX_SPLITS / 32; ++k) {
+      const float f = l[k] > 0.f ? exp2f(m[k] - M) : 0.f;
+      factor[lane + 32 * k] = f;
+      L += l[k] * f;
+    }
+    L = warp_sum(L);
+    if (sinks) L += exp2f(sinks[h] * LD_LOG2E - M);
+    if (lane == 0) s_inv = L > 0.f ? 1.f / L : 0.f;
+  }
+  __syncthreads();
+  const float inv = s_inv;
+  const int r4 = rank >> 2;                             // rank is a multiple of 8
+  const float4* src = reinterpret_cast<const float4*>(part_o) + base * r4;
+  for (int c = threadIdx.x; c < r4; c += blockDim.x) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i0 = 0; i0 < n_splits; i0 += 8) {
+      float4 t[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) t[j] = __ldcg(src + (size_t)min(i0 + j, n_splits - 1) * r4 + c);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float f = i0 + j < n_splits ? factor[i0 + j] : 0.f;
+        if (f == 0.f) continue;                         // a split without a key has written no columns
+        acc.x = fmaf(t[j].x, f, acc.x); acc.y = fmaf(t[j].y, f, acc.y);
+        acc.z = fmaf(t[j].z, f, acc.z); acc.w = fmaf(t[j].w, f, acc.w);
+      }
+    }
+    uint2 w;
+    w.x = ld_pack(acc.x * inv, acc.y * inv);
+    w.y = ld_pack(acc.z * inv, acc.w * inv);
+    *reinterpret_cast<uint2*>(out + (size_t)tok * out_stride + (size_t)h * rank + 4 * c) = w;
   }
 }
 
@@ -309,8 +345,9 @@ NHV_API int nhv_latent_decode(void* out, int out_stride, const void* q, int q_st
                               const float* sinks, int n_splits, float* part_o, float* part_ml, cudaStream_t stream) {
   if (n_tokens == 0 || n_seqs == 0) return 0;
   NHV_REQUIRE(nhv_latent_decode_supports(H, rank, row), "latent_decode: %d heads, a latent of %d in rows of %d: not taken", H, rank, row);
-  NHV_REQUIRE(n_splits > 0 && page_size > 0 && n_pages > 0 && bt_stride > 0 && q_stride % 8 == 0 &&
-              ((uintptr_t)q & 15) == 0 && ((uintptr_t)pages & 15) == 0, "latent_decode: bad geometry or alignment");
+  NHV_REQUIRE(n_splits > 0 && n_splits <= LD_MAX_SPLITS && page_size > 0 && n_pages > 0 && bt_stride > 0 && q_stride % 8 == 0 &&
+              ((uintptr_t)q & 15) == 0 && ((uintptr_t)pages & 15) == 0 && out_stride % 4 == 0 && ((uintptr_t)out & 7) == 0 &&
+              ((uintptr_t)part_o & 15) == 0 && ((uintptr_t)part_ml & 7) == 0, "latent_decode: bad geometry or alignment");
   const int RS = (row + 15) / 16 * 16 + 8;
   const size_t smem = (size_t)((16 + 2 * LD_BN) * RS + 16 * LD_PS) * sizeof(bf16) + (LD_WARPS * 16 + LD_KG * 32 * 4) * sizeof(float);
   dim3 grid(n_splits, n_tokens, (H + 15) / 16);

@@ -76,6 +76,34 @@ __global__ void latent_assemble_kernel(T* __restrict__ tmp, T* __restrict__ qp, 
   }
 }
 
+// The same in pieces of 8 elements, one block per temporary row or token (sizes and strides in steps of 8).  What lies in a
+// value row behind dv is not written: no column of the attention kernels' output that anyone reads depends on it.
+__global__ void latent_assemble_vec_kernel(uint4* __restrict__ tmp, uint4* __restrict__ qp, const uint4* __restrict__ kv,
+                                           const uint4* __restrict__ kr, const uint4* __restrict__ q, int q_stride,
+                                           const uint4* __restrict__ q_lat, int q_lat_stride, int n_rows, int H, int dn, int dr,
+                                           int dv, int rank, int D) {     // all in pieces
+  pdl_prologue();
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  if ((int)blockIdx.x < n_rows) {
+    const size_t r = blockIdx.x, page = r / LE_TILE, slot = r - page * LE_TILE;
+    const int per = D + dv;
+    const uint4* kvr = kv + r * (size_t)(H * (dn + dv));
+    for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+      const int h = i / per, c = i - h * per;
+      const int plane = c >= D, cc = plane ? c - D : c;
+      const uint4 v = plane ? kvr[H * dn + h * dv + cc] : (cc < dn ? kvr[h * dn + cc] : (cc < dn + dr ? kr[r * dr + cc - dn] : zero));
+      tmp[(((page * 2 + plane) * H + h) * LE_TILE + slot) * D + cc] = v;
+    }
+  } else {
+    const size_t t = blockIdx.x - n_rows;
+    for (int i = threadIdx.x; i < H * D; i += blockDim.x) {
+      const int h = i / D, c = i - h * D;
+      qp[t * (size_t)(H * D) + i] = c < dn ? q[t * q_stride + h * (dn + dr) + c]
+                                           : (c < dn + dr ? q_lat[t * q_lat_stride + h * (rank + dr) + rank + c - dn] : zero);
+    }
+  }
+}
+
 NHV_API int nhv_latent_gather(int dtype, void* lat, void* kr, const void* pages, const int* block_table, int bt_stride,
                               const int* kv_len, const int* row0, const int* first, int n_seqs, int max_rows, int rank, int dr, int row,
                               int page_size, int n_pages, cudaStream_t stream) {
@@ -102,6 +130,17 @@ NHV_API int nhv_latent_assemble(int dtype, void* tmp, void* qp, const void* kv, 
   if (n_rows == 0 && n_tokens == 0) return 0;
   NHV_REQUIRE(H > 0 && dn >= 0 && dr >= 0 && dv > 0 && D >= dn + dr && D >= dv && n_rows % LE_TILE == 0,
               "latent_assemble: a padded head of %d elements must hold the key's %d and the value's %d", D, dn + dr, dv);
+  auto on16 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+  if (dtype == NHV_BF16 && dn % 8 == 0 && dr % 8 == 0 && dv % 8 == 0 && rank % 8 == 0 && D % 8 == 0 && q_stride % 8 == 0 &&
+      q_lat_stride % 8 == 0 && on16(tmp) && on16(qp) && on16(kv) && on16(kr) && on16(q) && on16(q_lat) &&
+      n_rows + n_tokens < (1L << 31)) {
+    const int pieces = H * (D + dv) / 8;
+    nhv_launch(latent_assemble_vec_kernel, dim3((unsigned)(n_rows + n_tokens)), dim3(pieces >= 256 ? 256 : 64), 0, stream, (uint4*)tmp,
+               (uint4*)qp, (const uint4*)kv, (const uint4*)kr, (const uint4*)q, q_stride / 8, (const uint4*)q_lat, q_lat_stride / 8,
+               (int)n_rows, H, dn / 8, dr / 8, dv / 8, rank / 8, D / 8);
+    NHV_CHECK_LAUNCH("latent_assemble");
+    return 0;
+  }
   const size_t total = (2 * (size_t)n_rows + (size_t)n_tokens) * H * D;
   const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
 #define LAUNCH(T)                                                                                                    \

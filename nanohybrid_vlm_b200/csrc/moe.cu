@@ -20,6 +20,8 @@
 //   moe_combine   out[t] = sum_k w[t,k] * (choice is an expert ? y[row(t,k)] : x[t]) + sigmoid(sg[t]) * shared[t];
 //                 without weights every choice counts fully (the weights went into the experts' inputs).
 //
+// x of moe_combine may be null where no choice can be an identity expert.
+//
 // A row's result does not depend on where in its expert's run it stands, so the order in which moe_align hands out
 // rows (atomics) does not show in the numbers.
 #include <math.h>
@@ -330,16 +332,17 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y,
   float sg = 0.f;
   if (shared) sg = shared_gate ? 1.0f / (1.0f + expf(-shared_gate[(size_t)t * gate_stride])) : 1.0f;
   if constexpr (VEC) {
-    for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < width; c += gridDim.y * blockDim.x * 8) {
       float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, xv[8], v[8];
-      nhv_load8(xv, x + (size_t)t * width + c);
+      if (x) nhv_load8(xv, x + (size_t)t * width + c);          // null: no choice is an identity expert
+#pragma unroll 4
       for (int k = 0; k < top; ++k) {
         const int p = pos[k];
         if (p >= 0) {
           nhv_load8(v, y + (size_t)p * width + c);
 #pragma unroll
           for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[k], v[i], acc[i]);
-        } else if (p == -2) {
+        } else if (p == -2 && x) {
 #pragma unroll
           for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[k], xv[i], acc[i]);
         }
@@ -352,9 +355,9 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y,
       nhv_store8(out + (size_t)t * width + c, acc);
     }
   } else {
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
       float acc = 0.f;
-      const float xv = to_f32<T>(x[(size_t)t * width + c]);
+      const float xv = x ? to_f32<T>(x[(size_t)t * width + c]) : 0.f;
       for (int k = 0; k < top; ++k) {
         const int p = pos[k];
         if (p >= 0) acc = fmaf(w[k], to_f32<T>(y[(size_t)p * width + c]), acc);
@@ -373,10 +376,13 @@ NHV_API int nhv_moe_combine(int dtype, void* out, const void* y, const void* x, 
   NHV_REQUIRE(top > 0 && top <= 1024 && width > 0, "moe_combine: bad sizes");
   const bool vec = width % 8 == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)x % 16) == 0 &&
                    ((uintptr_t)shared % 16) == 0;
-  const int threads = vec ? (width >= 2048 ? 256 : 128) : (width >= 1024 ? 256 : 128);
+  const int threads = vec ? (width >= 2048 && n_tokens >= 148 ? 256 : 128) : (width >= 1024 ? 256 : 128);
   const size_t smem = (size_t)top * 8;
+  // few tokens: the columns of a token over several blocks, one piece a thread
+  const int spread = n_tokens < 148 ? (width + threads * (vec ? 8 : 1) - 1) / (threads * (vec ? 8 : 1)) : 1;
+  const dim3 grid(n_tokens, spread);
 #define GO(T, V)                                                                                                 \
-  nhv_launch(moe_combine_kernel<T, V>, n_tokens, threads, smem, stream, (T*)out, (const T*)y, (const T*)x, (const T*)shared, \
+  nhv_launch(moe_combine_kernel<T, V>, grid, threads, smem, stream, (T*)out, (const T*)y, (const T*)x, (const T*)shared, \
              shared_gate, gate_stride, ids, weights, slot_pos, top, E, width)
   if (dtype == NHV_F32) { if (vec) GO(float, true); else GO(float, false); }
   else if (dtype == NHV_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }

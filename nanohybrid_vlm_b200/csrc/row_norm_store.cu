@@ -1,7 +1,7 @@
 // Queries and keys normed over their whole projection (all heads of a kind together), optionally rotated, and the
 // key / value store, with values that may be mixed with the values of an earlier layer.
 //
-// One block per token of the packed projection output qkv [T, nq*dk + nkv*dk + nkv*dv]:
+// One block per token (its row is read once for the sums and once more, from the caches, for what is stored) of the packed projection output qkv [T, nq*dk + nkv*dk + nkv*dv]:
 //   q row [nq*dk]: x / sqrt(mean(x^2) + eps) * q_weight [nq*dk], then the rotation per head -> q_out [T, nq, q_head],
 //                  q_head >= dk, zeros behind a head's dk elements
 //   k row:         the same with k_weight [nkv*dk] -> the token's slot of the K pages
@@ -24,16 +24,15 @@ template <typename T> struct RowPiece<T, 1> {
   static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { *p = from_f32<T>(v[0]); }
 };
 
-template <typename T, int V>
-__global__ void row_norm_store_kernel(const T* __restrict__ qkv, int qkv_stride, T* __restrict__ q_out, int q_out_stride,
+template <typename T, int V, bool ROT>
+__global__ void __launch_bounds__(512, V == 8 && !ROT ? 3 : 1) row_norm_store_kernel(const T* __restrict__ qkv, int qkv_stride, T* __restrict__ q_out, int q_out_stride,
                                       int q_head, T* __restrict__ kv_pages, const int* __restrict__ slot_mapping,
                                       const int* __restrict__ positions, const float* __restrict__ cos_sin, int rotary_dim,
                                       int max_position, int interleaved, int nq, int nkv, int dk, int dv, int row,
                                       int page_size, int n_pages, float eps, const T* __restrict__ q_weight,
                                       const T* __restrict__ k_weight, const T* __restrict__ v_first, int v_first_stride,
                                       const float* __restrict__ v_share) {
-  extern __shared__ __align__(16) float buf[];              // the q row, then the k row
-  __shared__ float red[33];
+  __shared__ float2 red[33];
   pdl_prologue();
   const int t = blockIdx.x, nqd = nq * dk, nkd = nkv * dk;
   const T* src = qkv + (size_t)t * qkv_stride;
@@ -42,32 +41,30 @@ __global__ void row_norm_store_kernel(const T* __restrict__ qkv, int qkv_stride,
     slot = slot_mapping[t];
     if (slot >= n_pages * page_size) slot = -1;
   }
-  const int n_norm = slot >= 0 ? nqd + nkd : nqd;
-  float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x * V; c < n_norm; c += blockDim.x * V) {
-    float x[V];
-    RowPiece<T, V>::load(x, src + c);
-    float s = 0.f;
-#pragma unroll
-    for (int i = 0; i < V; ++i) s = fmaf(x[i], x[i], s);
-    if (c < nqd) sq += s; else sk += s;                      // V divides dk: a piece lies in one row
-    if (V == 8) {
-      float4* b = reinterpret_cast<float4*>(buf + c);
-      b[0] = make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]);
-      b[1] = make_float4(x[4 % V], x[5 % V], x[6 % V], x[7 % V]);
-    } else {
-      buf[c] = x[0];
-    }
-  }
   float rq = 1.f, rk = 1.f;
   if (eps >= 0.f) {
-    rq = 1.0f / sqrtf(block_sum(sq, red) / (float)nqd + eps);
-    rk = 1.0f / sqrtf(block_sum(sk, red) / (float)nkd + eps);
+    const int n_norm = slot >= 0 ? nqd + nkd : nqd;
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x * V; c < n_norm; c += blockDim.x * V) {
+      float x[V];
+      RowPiece<T, V>::load(x, src + c);
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < V; ++i) s = fmaf(x[i], x[i], s);
+      if (c < nqd) sq += s; else sk += s;                    // V divides dk: a piece lies in one row
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    if (lane == 0) red[warp] = make_float2(sq, sk);
+    __syncthreads();
+    float2 both = lane < n_warps ? red[lane] : make_float2(0.f, 0.f);     // every warp sums the warps' sums for itself
+    rq = 1.0f / sqrtf(warp_sum(both.x) / (float)nqd + eps);
+    rk = 1.0f / sqrtf(warp_sum(both.y) / (float)nkd + eps);
   }
-  __syncthreads();
   const float* cs = nullptr;
   const int half = rotary_dim >> 1;
-  if (cos_sin) {
+  if (ROT && cos_sin) {
     int pos = positions[t];
     pos = pos < 0 ? 0 : (pos >= max_position ? max_position - 1 : pos);
     cs = cos_sin + (size_t)pos * rotary_dim;                 // cos[0..half) then sin[0..half)
@@ -89,18 +86,20 @@ __global__ void row_norm_store_kernel(const T* __restrict__ qkv, int qkv_stride,
     for (int k = 0; k < V; ++k) o[k] = 0.f;
     if (kind < 2) {
       if (c0 < dk) {
-        const float* h = buf + (kind == 0 ? 0 : nqd) + head * dk;
+        const T* h = src + (kind == 0 ? 0 : nqd) + head * dk;
         const T* hw = eps >= 0.f ? (kind == 0 ? q_weight : k_weight) : nullptr;
         if (hw) hw += head * dk;
         const float r = kind == 0 ? rq : rk;
-        auto normed = [&](int c) { return hw ? h[c] * r * to_f32<T>(hw[c]) : h[c] * r; };
+        auto normed = [&](int c) { return hw ? to_f32<T>(h[c]) * r * to_f32<T>(hw[c]) : to_f32<T>(h[c]) * r; };
+        float x[V];
+        RowPiece<T, V>::load(x, h + c0);
         float wv[V];
         if (hw) RowPiece<T, V>::load(wv, hw + c0);
 #pragma unroll
         for (int k = 0; k < V; ++k) {
           const int c = c0 + k;
-          float v = hw ? h[c] * r * wv[k] : h[c] * r;
-          if (cs && c < rotary_dim) {
+          float v = hw ? x[k] * r * wv[k] : x[k] * r;
+          if (ROT && cs && c < rotary_dim) {
             if (interleaved) {
               const int a = c >> 1;
               v = (c & 1) ? v * cs[a] + normed(c - 1) * cs[half + a] : v * cs[a] - normed(c + 1) * cs[half + a];
@@ -138,30 +137,27 @@ NHV_API int nhv_row_norm_store(int dtype, const void* qkv, int qkv_stride, void*
   NHV_REQUIRE(kv_pages == nullptr || (page_size > 0 && n_pages > 0 && slot_mapping && row >= dk && row >= dv),
               "row_norm_store: a key/value store needs pages whose rows hold a head, and a slot mapping");
   NHV_REQUIRE(!v_first || v_share, "row_norm_store: mixed values need their share");
-  const size_t smem = (size_t)(nq + nkv) * dk * sizeof(float);
-  NHV_REQUIRE(smem <= 200 * 1024, "row_norm_store: %d query and key columns are beyond the %d a block holds", (nq + nkv) * dk, 200 * 1024 / 4);
   const int item = dtype == NHV_F32 ? 4 : 2;
-  auto on8 = [&](const void* p) { return ((uintptr_t)p % (dtype == NHV_F32 ? 16 : 16)) == 0; };
+  auto on8 = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
   const bool vec = dk % 8 == 0 && dv % 8 == 0 && q_head % 8 == 0 && row % 8 == 0 && (size_t)qkv_stride * item % 16 == 0 &&
                    (size_t)q_out_stride * item % 16 == 0 && (size_t)v_first_stride * item % 16 == 0 && on8(qkv) && on8(q_out) &&
                    on8(kv_pages) && on8(q_weight) && on8(k_weight) && on8(v_first);
   const int work = ((nq + nkv) * dk) / (vec ? 8 : 1);
   int threads = 64;
-  while (threads < 512 && threads < work) threads <<= 1;
-#define GO(T, V)                                                                                                      \
+  while (threads < (n_tokens <= 148 ? 512 : 256) && threads < work) threads <<= 1;
+#define GO2(T, V, R)                                                                                                    \
   do {                                                                                                                \
-    if (smem > 48 * 1024)                                                                                             \
-      NHV_CUDA(cudaFuncSetAttribute(row_norm_store_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), \
-               "row_norm_store");                                                                                     \
-    nhv_launch(row_norm_store_kernel<T, V>, n_tokens, threads, smem, stream, (const T*)qkv, qkv_stride, (T*)q_out,    \
+    nhv_launch(row_norm_store_kernel<T, V, R>, n_tokens, threads, 0, stream, (const T*)qkv, qkv_stride, (T*)q_out,    \
                q_out_stride, q_head, (T*)kv_pages, slot_mapping, positions, cos_sin, rotary_dim, max_position,        \
                interleaved, nq, nkv, dk, dv, row, page_size, n_pages, eps, (const T*)q_weight, (const T*)k_weight,    \
                (const T*)v_first, v_first_stride, v_share);                                                           \
   } while (0)
+#define GO(T, V) do { if (cos_sin) GO2(T, V, true); else GO2(T, V, false); } while (0)
   if (dtype == NHV_F32) { if (vec) GO(float, 8); else GO(float, 1); }
   else if (dtype == NHV_BF16) { if (vec) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
   else NHV_REQUIRE(false, "row_norm_store: unknown dtype %d", dtype);
 #undef GO
+#undef GO2
   NHV_CHECK_LAUNCH("row_norm_store");
   return 0;
 }

@@ -9,8 +9,9 @@
 //                      by the root mean square of its own elements
 // One block per row; the row of fp32 sums lives in shared memory between the two passes.
 #include "nhv_common.cuh"
+#include "nhv_vec8.cuh"
 
-template <typename T>
+template <typename T, bool VEC>
 __global__ void embed_scaled_f32_kernel(float* __restrict__ out, const T* __restrict__ table,
                                         const int* __restrict__ ids, int width, int vocab, float scale) {
   pdl_prologue();
@@ -19,7 +20,17 @@ __global__ void embed_scaled_f32_kernel(float* __restrict__ out, const T* __rest
   const bool ok = id >= 0 && id < vocab;
   const T* src = table + (size_t)(ok ? id : 0) * width;
   float* dst = out + (size_t)t * width;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = ok ? to_f32<T>(src[c]) * scale : 0.f;
+  if constexpr (VEC) {
+    for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+      float v[8];
+      nhv_load8(v, src + c);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[i] = ok ? v[i] * scale : 0.f;
+      nhv_store8(dst + c, v);
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = ok ? to_f32<T>(src[c]) * scale : 0.f;
+  }
 }
 
 NHV_API int nhv_embed_scaled_f32(int dtype, float* out, const void* table, const int* ids, int n_tokens, int width,
@@ -27,11 +38,12 @@ NHV_API int nhv_embed_scaled_f32(int dtype, float* out, const void* table, const
   if (n_tokens == 0) return 0;
   NHV_REQUIRE(n_tokens > 0 && width > 0 && vocab > 0, "embed_scaled_f32: bad sizes");
   const int threads = width >= 1024 ? 256 : 128;
-  if (dtype == NHV_F32)
-    nhv_launch(embed_scaled_f32_kernel<float>, n_tokens, threads, 0, stream, out, (const float*)table, ids, width, vocab, scale);
-  else if (dtype == NHV_BF16)
-    nhv_launch(embed_scaled_f32_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, out, (const __nv_bfloat16*)table, ids,
-               width, vocab, scale);
+  const bool vec = width % 8 == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)table % 16) == 0;
+#define GO(T, V) \
+  nhv_launch(embed_scaled_f32_kernel<T, V>, n_tokens, threads, 0, stream, out, (const T*)table, ids, width, vocab, scale)
+  if (dtype == NHV_F32) { if (vec) GO(float, true); else GO(float, false); }
+  else if (dtype == NHV_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
+#undef GO
   else
     NHV_REQUIRE(false, "embed_scaled_f32: unknown dtype %d", dtype);
   NHV_CHECK_LAUNCH("embed_scaled_f32");

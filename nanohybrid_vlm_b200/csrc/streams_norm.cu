@@ -137,7 +137,8 @@ NHV_API int nhv_streams_rmsnorm(int dtype, void* out, float* dst, const float* s
   const bool vec = width % 4 == 0 && ((uintptr_t)out % (4 * item)) == 0 && ((uintptr_t)dst % 16) == 0 && ((uintptr_t)src % 16) == 0 &&
                    ((uintptr_t)y % (4 * item)) == 0 && ((uintptr_t)w % (4 * item)) == 0;
   const int per = vec && n_streams <= 8 ? 4 : 1;
-  const int most = n_streams <= 8 && (vec || n_streams <= 4) ? 512 : 256;
+  // registers for the matrix and the copies leave few threads an SM: many small blocks where there are many rows
+  const int most = n_rows <= 148 && n_streams <= 8 && (vec || n_streams <= 4) ? 512 : 256;
   int threads = 32;
   while (threads < most && threads * per < width) threads <<= 1;
 #define GO(T, S, V)                                                                                                  \

@@ -14,7 +14,7 @@
 //
 // Warp roles.  Warp 0, one lane: TMA producer; per tile one box of 64 keys x 64 columns per 64 columns of the
 // head, for K and for V, from the pool seen as a matrix [pages * 2 * kv_heads * page_size, D], into two stages
-// each.  Warp 1: allocates tensor memory; one lane issues the MMAs: S = Q K^T (M 128, N 64, K = D; Q and K both
+// each (one stage of V where two would leave room for one block an SM only).  Warp 1: allocates tensor memory; one lane issues the MMAs: S = Q K^T (M 128, N 64, K = D; Q and K both
 // K-major in the 128-byte swizzle) into one of two S buffers, and O += P V (M 128, N = D, K = 64; P read from
 // tensor memory, V as it lies in the cache: MN-major).  Warps 2-5: one thread per row; it reads its row of S from
 // tensor memory, scales, masks, keeps the running maximum and sum, writes the row of P (bfloat16 pairs) over the
@@ -61,10 +61,16 @@ constexpr int Q_BYTES = DB * BM * 128;
 constexpr int T_BYTES = DB * BN * 128, V_BYTES = VB * BN * 128;     // one K tile, one V tile
 constexpr int STAGES = 2;
 constexpr int BAR_BYTES = 128;
-constexpr int SMEM_NEED = 1024 + Q_BYTES + STAGES * (T_BYTES + V_BYTES);    // barriers live in the first 128 bytes
+constexpr uint32_t TMEM_COLS = (2 * BN + DV) <= 256 ? 256 : 512;
+// Two blocks an SM: while one is in its softmax the other's products run.  Where tensor memory allows it and a single
+// stage of V makes it fit (an SM has 228 KB, a block takes 1 KB beside its own), V has one stage: the copy of a tile's V
+// then waits for the product of the tile before it and has that tile's softmax to arrive in.
+constexpr int smem_need(int v_stages) { return 1024 + Q_BYTES + STAGES * T_BYTES + v_stages * V_BYTES; }
+constexpr bool fits_twice(int v_stages) { return TMEM_COLS == 256 && 2 * (smem_need(v_stages) + 1024) <= 228 * 1024; }
+constexpr int V_STAGES = !fits_twice(2) && fits_twice(1) ? 1 : 2;
+constexpr int SMEM_NEED = smem_need(V_STAGES);    // barriers live in the first 128 bytes
 // at least 80 KB, so that an SM never holds more blocks than its tensor memory serves (two of 256 columns)
 constexpr int SMEM_BYTES = SMEM_NEED < 80 * 1024 ? 80 * 1024 : SMEM_NEED;
-constexpr uint32_t TMEM_COLS = (2 * BN + DV) <= 256 ? 256 : 512;
 constexpr uint32_t S_COL = 0, O_COL = 2 * BN;
 constexpr float RESCALE_STEP = 8.0f;         // log2 units
 constexpr float LOG2E = 1.4426950408889634f;
@@ -193,7 +199,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tc
   unsigned char* tiles = smem_raw + (((raw + BAR_BYTES + 1023u) & ~1023u) - raw);
   unsigned char* q_s = tiles;
   unsigned char* k_s = q_s + Q_BYTES;                  // [STAGES][T_BYTES]
-  unsigned char* v_s = k_s + STAGES * T_BYTES;         // [STAGES][V_BYTES]
+  unsigned char* v_s = k_s + STAGES * T_BYTES;         // [V_STAGES][V_BYTES]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -266,32 +272,44 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tc
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0 && n_tiles > 0) {
       const int* bt = p.block_table + (size_t)seq * p.bt_stride;
-      int issued = 0;
-      int page = bt[tile_key(0) / p.page_size];
-      for (int j = 0; j < n_tiles; ++j) {
+      int sent_k = 0, sent_v = 0;
+      auto row_of = [&](int j, int page) { return ((page * 2) * p.nkv + kvh) * p.page_size + tile_key(j) % p.page_size; };
+      auto send_k = [&](int j, int row) -> bool {
         const int st = j & 1;
-        const int key_base = tile_key(j);
-        int page_next = 0;
-        if (j + 1 < n_tiles) page_next = bt[tile_key(j + 1) / p.page_size];      // looked up one tile ahead
-        const int row_k = ((page * 2) * p.nkv + kvh) * p.page_size + key_base % p.page_size;
-        const int row_v = row_k + p.nkv * p.page_size;
-        if (j >= STAGES && !mbar_wait(&k_empty[st], (uint32_t)((j >> 1) - 1) & 1, 1)) { *s_abort = 1; break; }
+        if (j >= STAGES && !mbar_wait(&k_empty[st], (uint32_t)((j >> 1) - 1) & 1, 1)) return false;
         mbar_expect_tx(&k_full[st], T_BYTES);
 #pragma unroll
-        for (int b = 0; b < DB; ++b) tma_load_2d(k_s + st * T_BYTES + b * (BN * 128), &p.kv_map, b * 64, row_k, &k_full[st]);
-        if (j >= STAGES && !mbar_wait(&v_empty[st], (uint32_t)((j >> 1) - 1) & 1, 2)) { *s_abort = 1; issued = j; break; }
+        for (int b = 0; b < DB; ++b) tma_load_2d(k_s + st * T_BYTES + b * (BN * 128), &p.kv_map, b * 64, row, &k_full[st]);
+        sent_k = j + 1;
+        return true;
+      };
+      auto send_v = [&](int j, int row) -> bool {
+        const int st = j % V_STAGES;
+        if (j >= V_STAGES && !mbar_wait(&v_empty[st], (uint32_t)(j / V_STAGES - 1) & 1, 2)) return false;
         mbar_expect_tx(&v_full[st], V_BYTES);
 #pragma unroll
-        for (int b = 0; b < VB; ++b) tma_load_2d(v_s + st * V_BYTES + b * (BN * 128), &p.kv_map, b * 64, row_v, &v_full[st]);
-        issued = j + 1;
+        for (int b = 0; b < VB; ++b) tma_load_2d(v_s + st * V_BYTES + b * (BN * 128), &p.kv_map, b * 64, row, &v_full[st]);
+        sent_v = j + 1;
+        return true;
+      };
+      int page = bt[tile_key(0) / p.page_size];
+      bool sent = true;
+      if (V_STAGES == 1) sent = send_k(0, row_of(0, page));
+      for (int j = 0; j < n_tiles && sent; ++j) {
+        int page_next = 0;
+        if (j + 1 < n_tiles) page_next = bt[tile_key(j + 1) / p.page_size];      // looked up one tile ahead
+        const int row_k = row_of(j, page);
+        // with one stage of V the next tile's K goes ahead of this tile's V, which has a product to wait for
+        if (V_STAGES == 2) sent = send_k(j, row_k);
+        else if (j + 1 < n_tiles) sent = send_k(j + 1, row_of(j + 1, page_next));
+        if (sent) sent = send_v(j, row_k + p.nkv * p.page_size);
         page = page_next;
       }
-      if (*s_abort) {
-        // leave only when the copies in flight have landed: the last two tiles' barriers cover them
-        for (int j = max(0, issued - STAGES); j < issued; ++j) {
-          mbar_wait(&k_full[j & 1], (uint32_t)(j >> 1) & 1, 3);
-          mbar_wait(&v_full[j & 1], (uint32_t)(j >> 1) & 1, 3);
-        }
+      if (!sent) {
+        *s_abort = 1;
+        // leave only when the copies in flight have landed: the last stages' barriers cover them
+        for (int j = max(0, sent_k - STAGES); j < sent_k; ++j) mbar_wait(&k_full[j & 1], (uint32_t)(j >> 1) & 1, 3);
+        for (int j = max(0, sent_v - V_STAGES); j < sent_v; ++j) mbar_wait(&v_full[j % V_STAGES], (uint32_t)(j / V_STAGES) & 1, 3);
       }
     }
     __syncwarp();
@@ -322,19 +340,19 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tc
       };
       ok = issue_qk(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int st = j & 1;
+        const int sv = j % V_STAGES;
         if (j + 1 < n_tiles) ok = issue_qk(j + 1);
         if (!ok) break;
-        ok = mbar_wait(p_ready, (uint32_t)j & 1, 5) && mbar_wait(&v_full[st], (uint32_t)(j >> 1) & 1, 6);
+        ok = mbar_wait(p_ready, (uint32_t)j & 1, 5) && mbar_wait(&v_full[sv], (uint32_t)(j / V_STAGES) & 1, 6);
         if (!ok) break;
         tc_fence_after();
-        const uint64_t vd = v_desc + (uint64_t)(st * (V_BYTES >> 4));
+        const uint64_t vd = v_desc + (uint64_t)(sv * (V_BYTES >> 4));
         const uint32_t p_addr = tmem_base + S_COL + (uint32_t)((j & 1) * BN);    // P lies over the first half of this tile's S
 #pragma unroll
         for (int kk = 0; kk < BN / 16; ++kk)                                       // 8 columns of P and 16 rows of V per 16 keys
           tc_mma_a_tmem(tmem_base + O_COL, p_addr + kk * 8, vd + (uint64_t)((kk * 16 * 128) >> 4), idesc_o,
                         (j > 0 || kk > 0) ? 1u : 0u);
-        tc_commit(&v_empty[st]);
+        tc_commit(&v_empty[sv]);
         tc_commit(o_full);
       }
       if (!ok) *s_abort = 1;
@@ -435,12 +453,12 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tc
       tmem_st_wait();
       if (key_base + BN > total) {
         // keys beyond the request's last one: their V rows may hold anything (0 * NaN = NaN), so zero them
-        ok = mbar_wait(&v_full[j & 1], (uint32_t)(j >> 1) & 1, 10);
+        ok = mbar_wait(&v_full[j % V_STAGES], (uint32_t)(j / V_STAGES) & 1, 10);
         if (!ok) break;
         const int first_bad = total - key_base;                  // 1..63
         for (int id = threadIdx.x - 64; id < (BN - first_bad) * VB * 8; id += 128) {
           const int row = first_bad + id / (VB * 8), rem = id % (VB * 8);
-          *reinterpret_cast<uint4*>(v_s + (j & 1) * V_BYTES + (rem >> 3) * (BN * 128) + row * 128 + ((rem & 7) << 4)) =
+          *reinterpret_cast<uint4*>(v_s + (j % V_STAGES) * V_BYTES + (rem >> 3) * (BN * 128) + row * 128 + ((rem & 7) << 4)) =
               make_uint4(0, 0, 0, 0);
         }
         fence_async_smem();

@@ -785,15 +785,17 @@ def _moe_experts_tcgen05(x, gate, up, down, ids, limit: float, alpha: float, up_
 def moe_combine(out, y, x, ids, weights, slot_pos, n_experts: int, shared=None, shared_gate=None) -> None:
     """out[t] = sum over the token's choices of weight * (the expert's row of y, or x[t] itself for an identity expert)
     (+ sigmoid(shared_gate[t]) * shared[t]; a shared term without a gate counts fully).  ``shared_gate``: a float32
-    column view (one number per token).  ``weights`` None: every choice counts fully."""
+    column view (one number per token).  ``weights`` None: every choice counts fully.  ``x`` None: no choice is an identity
+    expert."""
     _need_cuda(out, y, x, ids, weights, slot_pos, shared, shared_gate)
-    _contig("out", out); _contig("y", y); _contig("x", x)
-    T, width = x.shape
+    _contig("out", out); _contig("y", y)
+    T, width = out.shape
     top = ids.shape[1]
-    assert out.shape == x.shape and y.shape[1] == width and out.dtype == y.dtype == x.dtype
-    assert shared is None or (shared.shape == x.shape and shared.dtype == x.dtype and shared.is_contiguous())
+    assert y.shape[1] == width and out.dtype == y.dtype
+    assert x is None or (x.shape == out.shape and x.dtype == out.dtype and x.is_contiguous())
+    assert shared is None or (shared.shape == out.shape and shared.dtype == out.dtype and shared.is_contiguous())
     assert shared_gate is None or (shared is not None and shared_gate.dtype == torch.float32 and shared_gate.shape[0] == T)
-    call("nhv_moe_combine", dtype_code(out), out.data_ptr(), y.data_ptr(), x.data_ptr(), _ptr(shared), _ptr(shared_gate),
+    call("nhv_moe_combine", dtype_code(out), out.data_ptr(), y.data_ptr(), _ptr(x), _ptr(shared), _ptr(shared_gate),
          0 if shared_gate is None else shared_gate.stride(0), ids.data_ptr(), _ptr(weights), slot_pos.data_ptr(), T, top,
          n_experts, width, stream_ptr())
 
@@ -1450,7 +1452,7 @@ def linear_simt(out, x, weight) -> None:
 # leaves with whatever it has, so the step's results are not valid.  The words reach the host with the step's
 # tokens: the sampler folds them into one more int behind the tokens (``sample`` below), and callers that read
 # logits instead ask ``take_wait_errors`` once per step.
-ERROR_WORD_SLOTS = 16
+ERROR_WORD_SLOTS = 31
 _wait_error_sources: list = []          # (name, function giving the word's device address, function that reads and clears it)
 _error_word_arrays: dict = {}           # device -> (int64 tensor [ERROR_WORD_SLOTS] of addresses, sources filled in)
 

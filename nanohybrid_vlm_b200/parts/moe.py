@@ -132,6 +132,11 @@ class RoutedMoE(FeedForward):
     def bind(self, tensors):
         p = self.SHARED_PREFIX
         super().bind({n: t for n, t in tensors.items() if not n.startswith(p)})
+        # bfloat16: the router's rows padded with zeros to a multiple of 8, where the library product takes the step
+        self.router_rows = None
+        pad = -self.w_router.shape[0] % 8
+        if pad and self.w_router.dtype == torch.bfloat16:
+            self.router_rows = torch.cat([self.w_router, self.w_router.new_zeros(pad, self.w_router.shape[1])])
         if self.shared is not None:
             self.shared.bind({n[len(p):]: t for n, t in tensors.items() if n.startswith(p)})
 
@@ -140,8 +145,11 @@ class RoutedMoE(FeedForward):
 
     def forward(self, x, batch):
         T, W = x.shape
-        logits = self.new(T, self.N + int(self.shared_gate), dtype=torch.float32)
-        ops.linear_f32(logits, x, self.w_router)
+        router = self.w_router
+        if self.router_rows is not None and T * router.shape[0] > ops.LINEAR_F32_ROWS_LIMIT:
+            router = self.router_rows
+        logits = self.new(T, router.shape[0], dtype=torch.float32)
+        ops.linear_f32(logits, x, router)
         ids = self.new(T, self.top, dtype=torch.int32)
         weights = self.new(T, self.top, dtype=torch.float32)
         ops.moe_route(ids, weights, logits, self.w_correction if self.has_correction else None, self.N, self.groups, self.keep,
@@ -152,7 +160,7 @@ class RoutedMoE(FeedForward):
                                       weights if on_input else None)
         shared = self.shared.forward(x, batch) if self.shared is not None else None
         out = self.new(T, W)
-        ops.moe_combine(out, y, x, ids, None if on_input else weights, slot_pos, self.E, shared,
+        ops.moe_combine(out, y, x if self.I0 else None, ids, None if on_input else weights, slot_pos, self.E, shared,
                         logits[:, self.N] if self.shared_gate else None)
         return out
 
