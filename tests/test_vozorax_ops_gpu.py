@@ -96,7 +96,7 @@ def test_the_mixing_matrix_is_indexed_from_to(ops):
 def test_block_over_streams(dtype):
     """Two layers (the second without a feed-forward) of parts that compute simple things, the embedding as one row to
     start from, the last norm at some rows."""
-    from nanohybrid_vlm_b200.parts import CONNECTIONS, FEED_FORWARDS, NORMS, part
+    from nanohybrid_vlm_b200.parts import CONNECTIONS, NORMS, part
     from nanohybrid_vlm_b200.parts.base import BLOCKS
     S, W, T = 3, 40, 7
     g = torch.Generator().manual_seed(8)
@@ -133,7 +133,6 @@ def test_block_over_streams(dtype):
     close(got, (pv.unit_rms(X.sum(0), EPS) * nwf["norm1"])[rows], dtype)
     with pytest.raises(ValueError, match="connection"):
         cls(part("hyper_connections"), dict(mixer=Product(mats[0]), mixer_norm=n1, mixer_connection=c1, ffn=Product(mats[1])))
-    assert FEED_FORWARDS is not None
 
 
 # ---------------------------------------------------------------- latent attention in a window
@@ -184,12 +183,12 @@ def standing_out(T, H, dk, first, second):
 @pytest.mark.parametrize("portion", [1, 2, 30])
 def test_keys_just_inside_and_just_outside_a_latent_window(ops, dtype, window, portion):
     """Two keys outweigh all others; the later tokens see both, then one, then neither as the window passes them."""
+    from nanohybrid_vlm_b200.parts import PagedKVNeed
     H, rank, dr, page = 3, 32, 8, 16
     row, T = rank + dr, 240
     at = 70
     q, k = standing_out(T, H, row, at, at + 1)
-    k = k.clone()
-    rig = Rig([SimpleNamespaceNeed(row, window, rank)], page_size=page, num_pages=20, dtype=dtype)
+    rig = Rig([PagedKVNeed(1, row, window, v_head_dim=rank, planes=1)], page_size=page, num_pages=20, dtype=dtype)
     got, done = [], 0
     while done < T:
         n = min(portion if done >= 60 else 60, T - done)
@@ -210,11 +209,6 @@ def test_keys_just_inside_and_just_outside_a_latent_window(ops, dtype, window, p
     # the steps of the window show: both keys, the later one alone, neither
     a, b_, c = (got[at + window + i - 1, 0].item() for i in (0, 1, 2))
     assert c < 0.2 * b_ and abs(a - b_) > 0.005 * b_
-
-
-def SimpleNamespaceNeed(row, window, rank):
-    from nanohybrid_vlm_b200.parts import PagedKVNeed
-    return PagedKVNeed(1, row, window, v_head_dim=rank, planes=1)
 
 
 # ---------------------------------------------------------------- attention with rows normed whole and mixed values
