@@ -866,7 +866,10 @@ def bench_designs(args) -> dict:
                "prefill_ms": round(prefill_ms, 3),
                "prefill_tok_s": round(T / prefill_ms * 1e3),
                "prefill_us_by_kind": {k: round(v, 1) for k, v in sorted(by_kind.items(), key=lambda kv: -kv[1])}}
-        gemm_flops = 2.0 * T * (weights_2d - vocab * cfg.get("width", cfg.get("hidden_size")))
+        # the embedding is looked up, and a head multiplies the one row that is asked for
+        tables = sum(bp.decl.shape[0] * bp.decl.shape[1] for bp in runner.model.param_table()
+                     if len(bp.decl.shape) == 2 and bp.decl.shape[0] == vocab)
+        gemm_flops = 2.0 * T * (weights_2d - tables)
         if "gemm" in by_kind:
             out["gemm_frac_of_measured_bf16"] = round(gemm_flops / (by_kind["gemm"] * 1e-6) / (pk["bf16_tflops"] * 1e12), 3)
         if "experts" in by_kind:     # an upper bound of the work: every choice counted as a real expert
