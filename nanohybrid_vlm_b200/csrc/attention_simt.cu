@@ -25,6 +25,7 @@
 // Two more: a bias by distance, score - slopes[head] * (query position - key position), and pages with one plane
 // (planes == 1): a row of such a page is the key, and its leading dv elements are the value as well (keys and
 // values that are one latent vector per token, stored once).
+// A cap on the scores (softcap > 0): score <- softcap * tanh(score / softcap), before anything is added to it.
 // And kept first keys (keep_first, with a window): a query also sees the keys at positions below keep_first, at their
 // true positions; their chunks are visited before the window's.
 #include <math.h>
@@ -43,7 +44,8 @@ __global__ void attn_paged_simt_kernel(const T* __restrict__ q, int q_stride, T*
                                        int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ kv_len,
                                        int n_seqs, int nq, int nkv, int d, int page_size, int n_pages, int window,
                                        float scale, int TQ, int GS, int dv, int row, const float* __restrict__ sinks,
-                                       int chunk, const float* __restrict__ slopes, int planes, int keep_first) {
+                                       int chunk, const float* __restrict__ slopes, int planes, int keep_first,
+                                       float softcap) {
   extern __shared__ float smem[];
   constexpr int AT_COLS = COLS, AT_PAIRS_PER_WARP = AT_ACC / COLS, AT_MAX_PAIRS = AT_PAIRS_PER_WARP * AT_WARPS;
   pdl_prologue();
@@ -154,6 +156,7 @@ __global__ void attn_paged_simt_kernel(const T* __restrict__ q, int q_stride, T*
         float acc = 0.f;
         for (int c = 0; c < d; ++c) acc = fmaf(qv[c], kv[c], acc);
         s = acc * scale;
+        if (softcap > 0.f) s = softcap * tanhf(s / softcap);
         if (slopes) s -= slopes[kvh * G + g0 + (p - tq * gs)] * (float)(pos - j);
       }
       const float cmax = warp_max(s);
@@ -200,9 +203,10 @@ NHV_API int nhv_attention_simt_ex(int dtype, const void* q, int q_stride, void* 
                                   const void* kv_pages, const int* block_table, int bt_stride, const int* cu_q,
                                   const int* kv_len, int n_seqs, int n_tokens, int nq, int nkv, int d, int dv, int row,
                                   int page_size, int n_pages, int window, int chunk, float scale, const float* sinks,
-                                  const float* slopes, int planes, int keep_first, cudaStream_t stream) {
+                                  const float* slopes, int planes, int keep_first, float softcap, cudaStream_t stream) {
   if (n_tokens == 0 || n_seqs == 0) return 0;
   NHV_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention: kept first keys go with a window");
+  NHV_REQUIRE(softcap >= 0.f, "attention: a cap on the scores must be positive");
   NHV_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention: %d query heads do not divide into %d KV heads", nq, nkv);
   NHV_REQUIRE(d > 0 && d <= AT_MAX_D && dv > 0 && dv <= AT_MAX_D, "attention: head sizes %d / %d are beyond the supported %d",
               d, dv, AT_MAX_D);
@@ -227,7 +231,7 @@ NHV_API int nhv_attention_simt_ex(int dtype, const void* q, int q_stride, void* 
     nhv_launch(attn_paged_simt_kernel<T, COLS>, grid, AT_WARPS * 32, smem, stream,                                   \
         (const T*)q, q_stride, (T*)out, out_stride, (const T*)kv_pages, block_table, bt_stride, cu_q, kv_len,        \
         n_seqs, nq, nkv, d, page_size, n_pages, window, scale, TQ, GS, dv, row, sinks, chunk, slopes, planes,        \
-        keep_first);                                                                                                 \
+        keep_first, softcap);                                                                                        \
   } while (0)
 #define LAUNCH_COLS(T)                 \
   do {                                 \
@@ -250,5 +254,5 @@ NHV_API int nhv_attention_simt(int dtype, const void* q, int q_stride, void* out
                                const int* kv_len, int n_seqs, int n_tokens, int nq, int nkv, int d, int page_size,
                                int n_pages, int window, float scale, cudaStream_t stream) {
   return nhv_attention_simt_ex(dtype, q, q_stride, out, out_stride, kv_pages, block_table, bt_stride, cu_q, kv_len,
-                               n_seqs, n_tokens, nq, nkv, d, d, d, page_size, n_pages, window, 0, scale, nullptr, nullptr, 2, 0, stream);
+                               n_seqs, n_tokens, nq, nkv, d, d, d, page_size, n_pages, window, 0, scale, nullptr, nullptr, 2, 0, 0.f, stream);
 }

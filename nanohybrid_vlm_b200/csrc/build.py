@@ -16,6 +16,7 @@ import shutil
 import subprocess
 import sys
 import tempfile
+import threading
 import time
 
 CSRC = os.path.dirname(os.path.abspath(__file__))
@@ -56,7 +57,7 @@ def source_hash() -> str:
 def _writable_dir(path: str) -> bool:
     try:
         os.makedirs(path, exist_ok=True)
-        probe = os.path.join(path, f".probe{os.getpid()}")
+        probe = os.path.join(path, f".probe{os.getpid()}_{threading.get_ident()}")
         with open(probe, "w"):
             pass
         os.remove(probe)

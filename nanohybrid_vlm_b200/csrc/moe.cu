@@ -6,6 +6,8 @@
 //                 neighbours, a group's score is its largest c, and only outputs of the `keep` best groups can be
 //                 chosen (the others count as -inf); the `top` outputs with the largest c are chosen; their weights
 //                 are their s, divided by the sum of the chosen s (+ 1e-20).  One warp per token, all in fp32.
+//                 group_best 2: a group's score is the sum of its two largest c (of its one, where it has no more);
+//                 factor: multiplies the weights.
 //                 scores 1: s = sigmoid(z) instead of the softmax; renorm 0: the weights are the chosen s as they are.
 //                 scores 2: s = c = z + correction (a bias of the logits), and the weights are the softmax over the
 //                 chosen alone.
@@ -44,7 +46,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits, int ld,
     const float* __restrict__ correction, int n_tokens, int N, int n_groups, int keep, int top, int scores,
-    int renorm) {
+    int renorm, int group_best, float factor) {
   extern __shared__ float smem[];
   pdl_prologue();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -83,9 +85,13 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
   if (n_groups > 1 && keep < n_groups) {
     const int gsz = N / n_groups;
     for (int g = lane; g < n_groups; g += 32) {
-      float best = -INFINITY;
-      for (int j = 0; j < gsz; ++j) best = fmaxf(best, c[g * gsz + j]);
-      gs[g] = best;
+      float best = -INFINITY, second = -INFINITY;
+      for (int j = 0; j < gsz; ++j) {
+        const float v = c[g * gsz + j];
+        second = fmaxf(second, fminf(best, v));
+        best = fmaxf(best, v);
+      }
+      gs[g] = group_best == 2 && gsz > 1 ? best + second : best;
     }
     __syncwarp();
     for (int r = 0; r < keep; ++r) {
@@ -121,21 +127,23 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(
     wsum += w;
     if (lane == 0) {
       ids[(size_t)t * top + r] = bi;
-      weights[(size_t)t * top + r] = w;
+      weights[(size_t)t * top + r] = !renorm && scores != 2 ? w * factor : w;
       c[bi] = -INFINITY;
     }
     __syncwarp();
   }
   if (!renorm && scores != 2) return;
   __syncwarp();
-  const float inv = 1.0f / (wsum + (scores == 2 ? 0.f : 1e-20f));
+  const float inv = factor / (wsum + (scores == 2 ? 0.f : 1e-20f));
   for (int r = lane; r < top; r += 32) weights[(size_t)t * top + r] *= inv;
 }
 
 NHV_API int nhv_moe_route(int* ids, float* weights, const float* logits, int ld, const float* correction, int n_tokens, int N,
-                          int n_groups, int keep, int top, int scores, int renorm, cudaStream_t stream) {
+                          int n_groups, int keep, int top, int scores, int renorm, int group_best, float factor,
+                          cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   NHV_REQUIRE(N > 0 && N <= 4096 && top > 0 && top <= N && ld >= N, "moe_route: bad sizes (N %d, top %d)", N, top);
+  NHV_REQUIRE(group_best == 1 || group_best == 2, "moe_route: a group's score is its best choice score or the sum of its best two");
   NHV_REQUIRE(scores >= 0 && scores <= 2, "moe_route: unknown kind of scores %d", scores);
   NHV_REQUIRE(n_groups > 0 && N % n_groups == 0 && keep > 0 && keep <= n_groups,
               "moe_route: %d outputs do not form %d equal groups of which %d are kept", N, n_groups, keep);
@@ -144,7 +152,7 @@ NHV_API int nhv_moe_route(int* ids, float* weights, const float* logits, int ld,
   if (smem > 48 * 1024)
     NHV_CUDA(cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "moe_route");
   nhv_launch(moe_route_kernel, (n_tokens + MR_WARPS - 1) / MR_WARPS, MR_WARPS * 32, smem, stream, ids, weights, logits, ld,
-             correction, n_tokens, N, n_groups, keep, top, scores, renorm);
+             correction, n_tokens, N, n_groups, keep, top, scores, renorm, group_best, factor);
   NHV_CHECK_LAUNCH("moe_route");
   return 0;
 }

@@ -139,6 +139,34 @@ __host__ __device__ __forceinline__ int nhv_first_key(int pos, int window, int c
   return lo;
 }
 
+// Scores capped smoothly, cap * tanh(raw * scale / cap), in log2 units: cap * log2(e) * (1 - 2 / (1 + e^(2 z))) with
+// z = raw * scale / cap, so that exp2 of it is the exponential of the capped score.  `in` = 2 log2(e) scale / cap turns a
+// raw score into the exponent of 2, `out` = cap log2(e).  Two scores share one reciprocal (of the product of both
+// denominators, whose exponents are kept below 2^60 so that it cannot overflow: tanh is 1 to the last bit long before).
+// The error is a few units of 2^-24 of the cap.
+struct NhvScoreCap {
+  float in, out;      // in == 0: scores are not capped
+};
+inline NhvScoreCap nhv_score_cap(float scale, float cap) {
+  NhvScoreCap c = {0.f, 0.f};
+  if (cap > 0.f) {
+    c.in = 2.0f * 1.4426950408889634f * scale / cap;
+    c.out = cap * 1.4426950408889634f;
+  }
+  return c;
+}
+__device__ __forceinline__ void nhv_cap_scores(float& a, float& b, const NhvScoreCap& c) {
+  float ea, eb, r;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(ea) : "f"(fminf(a * c.in, 60.f)));
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(eb) : "f"(fminf(b * c.in, 60.f)));
+  ea += 1.f;
+  eb += 1.f;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(ea * eb));
+  r *= -2.0f * c.out;
+  a = fmaf(r, eb, c.out);
+  b = fmaf(r, ea, c.out);
+}
+
 template <typename T> __device__ __forceinline__ float to_f32(T v);
 template <> __device__ __forceinline__ float to_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }

@@ -211,7 +211,7 @@ struct RowState {
 // the kept first keys [0, keep_first).
 __device__ __forceinline__ void warp_half_tile(RowState& st, const uint32_t (&qf)[KS][4], const bf16* ks, const bf16* vs,
                                                int kb, int key_base, int lo, const int (&row_hi)[2], float scale_log2,
-                                               int keep_first) {
+                                               int keep_first, const NhvScoreCap& cap) {
   const int lane = threadIdx.x & 31;
   constexpr int NT = 4;
   float s[NT][4];
@@ -226,6 +226,13 @@ __device__ __forceinline__ void warp_half_tile(RowState& st, const uint32_t (&qf
       ldmatrix_x4(b, ks + tile_off<BN>(kb + 8 * j + (lane & 7) + ((lane >> 4) << 3), 2 * k + ((lane >> 3) & 1)));
       mma_bf16(s[j], qf[k], b[0], b[1]);
       mma_bf16(s[j + 1], qf[k], b[2], b[3]);
+    }
+  }
+  if (cap.in != 0.f) {                                         // capped scores are in log2 units: scale_log2 is 1 then
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      nhv_cap_scores(s[j][0], s[j][1], cap);
+      nhv_cap_scores(s[j][2], s[j][3], cap);
     }
   }
   float mx[2] = {-INFINITY, -INFINITY};
@@ -300,7 +307,8 @@ struct alignas(64) Params {
   int q_stride, out_stride, bt_stride, n_seqs, nq, nkv, page_size, n_pages, window, chunk;
   int out_head;             // elements between two heads of the output, up to DV: that many are written
   int keep_first;           // with a window: the keys at positions below it stay visible; their tiles come first
-  float scale_log2;
+  float scale_log2;         // 1 with capped scores, which are in log2 units already
+  NhvScoreCap cap;          // in == 0: none
   FusedQK fq;
 };
 
@@ -669,7 +677,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_decode_kernel(const __grid_co
       if (wrote) __syncwarp();
       const int lo_t = there ? lo : 0x7fffffff;               // a tile whose page is missing: no key counts
       if (key_base < total && (key_base + BN > lo_t || (there && key_base < keep_first)))
-        warp_half_tile(st, qf, kt, vt, 0, key_base, lo_t, row_hi, p.scale_log2, there ? keep_first : 0);
+        warp_half_tile(st, qf, kt, vt, 0, key_base, lo_t, row_hi, p.scale_log2, there ? keep_first : 0, p.cap);
       if (wrote) fence_async_smem();                          // this warp's stores before the next copy into the stage
       __syncwarp();
       if (lane == 0) mbar_arrive(&empty[stage]);
@@ -837,7 +845,8 @@ NHV_API int NHV_FN(nhv_attn_decode_d)(const void* q, int q_stride, const void* q
                                       int window, int chunk, float scale, float* part_o, float* part_ml, int* counters,
                                       const void* q_w, const void* k_w, const float* cos_sin, const int* positions,
                                       const int* slot_mapping, int rotary_dim, int max_position, int store, float eps,
-                                      float weight_offset, const float* sinks, int keep_first, int out_head, cudaStream_t stream) {
+                                      float weight_offset, const float* sinks, int keep_first, int out_head, float softcap,
+                                      cudaStream_t stream) {
   ATT_REQUIRE(out_head > 0 && out_head <= DV && out_head % 8 == 0,
               "attention (decode, TMA): an output head has %d elements, in steps of 8 up to %d", out_head, DV);
   ATT_REQUIRE(!qkv || (DV == D && out_head == D), "attention: the form that works from the projection has heads of one size");
@@ -924,7 +933,9 @@ NHV_API int NHV_FN(nhv_attn_decode_d)(const void* q, int q_stride, const void* q
   p.out_head = out_head;
   p.q_stride = q_stride; p.out_stride = out_stride; p.bt_stride = bt_stride; p.n_seqs = n_seqs; p.nq = nq; p.nkv = nkv;
   p.page_size = page_size; p.n_pages = n_pages; p.window = window; p.chunk = chunk; p.keep_first = keep_first;
-  p.scale_log2 = scale * LOG2E;
+  ATT_REQUIRE(softcap >= 0.f, "attention: a cap on the scores must be positive");
+  p.cap = nhv_score_cap(scale, softcap);
+  p.scale_log2 = softcap > 0.f ? 1.0f : scale * LOG2E;
   const cudaError_t launched = deep ? nhv_launch(attn_decode_kernel<STAGES_DEEP, 8>, dim3(blocks), dim3(THREADS), smem, stream, p)
                                     : nhv_launch(attn_decode_kernel<STAGES_MIN, 16>, dim3(blocks), dim3(THREADS), smem, stream, p);
   if (launched != cudaSuccess || cudaPeekAtLastError() != cudaSuccess) {

@@ -140,7 +140,8 @@ struct RowState {
 template <int NT>
 __device__ __forceinline__ void warp_tile(RowState& st, const uint32_t (&qf)[KS][4], const bf16* ks, const bf16* vs,
                                           int kb, int key_base, const int (&row_lo)[2], const int (&row_hi)[2],
-                                          float scale_log2, const float (&row_slope)[2], int keep_first) {
+                                          float scale_log2, const float (&row_slope)[2], int keep_first,
+                                          const NhvScoreCap& cap) {
   const int lane = threadIdx.x & 31;
   float s[NT][4];
 #pragma unroll
@@ -154,6 +155,13 @@ __device__ __forceinline__ void warp_tile(RowState& st, const uint32_t (&qf)[KS]
       ldmatrix_x4(b, ks + tile_off(kb + 8 * j + (lane & 7) + ((lane >> 4) << 3), 2 * k + ((lane >> 3) & 1)));
       mma_bf16(s[j], qf[k], b[0], b[1]);
       mma_bf16(s[j + 1], qf[k], b[2], b[3]);
+    }
+  }
+  if (cap.in != 0.f) {                                         // capped scores are in log2 units: scale_log2 is 1 then
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      nhv_cap_scores(s[j][0], s[j][1], cap);
+      nhv_cap_scores(s[j][2], s[j][3], cap);
     }
   }
   // mask and the tile's row maxima
@@ -246,7 +254,7 @@ template <int MTW>
 __device__ __forceinline__ void warp_tile_prefill(PrefillState<MTW>& st, const bf16* qs, int qrow0, const bf16* ks, const bf16* vs,
                                                   int key_base, const int (&row_lo)[MTW][2], const int (&row_hi)[MTW][2],
                                                   int w_lo, int w_hi, float scale_log2, const float (&row_slope)[MTW][2],
-                                                  int keep_first) {
+                                                  int keep_first, const NhvScoreCap& cap) {
   const int lane = threadIdx.x & 31;
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
@@ -274,6 +282,15 @@ __device__ __forceinline__ void warp_tile_prefill(PrefillState<MTW>& st, const b
           mma_bf16(s[mt][j + 1], a[mt], b[2], b[3]);
         }
       }
+    }
+    if (cap.in != 0.f) {
+#pragma unroll
+      for (int mt = 0; mt < MTW; ++mt)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          nhv_cap_scores(s[mt][j][0], s[mt][j][1], cap);
+          nhv_cap_scores(s[mt][j][2], s[mt][j][3], cap);
+        }
     }
     uint32_t pf[MTW][2][4];
 #pragma unroll
@@ -341,7 +358,7 @@ __global__ void __launch_bounds__(THREADS, MTW == 2 ? 2 : (D <= 128 ? 3 : 1)) at
     const bf16* __restrict__ kv_pages, const int* __restrict__ block_table, int bt_stride,
     const int* __restrict__ cu_q, const int* __restrict__ kv_len, int n_seqs, int nq, int nkv, int page_size,
     int n_pages, int window, int chunk, float scale_log2, int tokens_per_block, const float* __restrict__ sinks,
-    const float* __restrict__ slopes, int keep_first, int out_head) {
+    const float* __restrict__ slopes, int keep_first, int out_head, const NhvScoreCap cap) {
   constexpr int PF_ROWS = 64 * MTW;                          // rows (token x head of the group) per block
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qbuf = reinterpret_cast<bf16*>(smem_raw);            // [PF_ROWS rows]
@@ -438,7 +455,7 @@ __global__ void __launch_bounds__(THREADS, MTW == 2 ? 2 : (D <= 128 ? 3 : 1)) at
     const int key_base = tile_key(it);
     if (key_base <= w_hi && (key_base + BN > w_lo || key_base < keep_first))
       warp_tile_prefill<MTW>(st, qbuf, warp * WROWS, kbuf + stage * TILE_ELEMS, vbuf + stage * TILE_ELEMS, key_base, row_lo,
-                        row_hi, w_lo, w_hi, scale_log2, row_slope, keep_first);
+                        row_hi, w_lo, w_hi, scale_log2, row_slope, keep_first, cap);
     __syncthreads();
   }
 #pragma unroll
@@ -538,7 +555,7 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
     const int* __restrict__ block_table, int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ kv_len,
     float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int n_seqs, int nq, int nkv,
     int page_size, int n_pages, int window, int chunk, float scale_log2, int max_pieces, const FusedQK fq,
-    const float* __restrict__ sinks, const float* __restrict__ slopes, int keep_first, int out_head) {
+    const float* __restrict__ sinks, const float* __restrict__ slopes, int keep_first, int out_head, const NhvScoreCap cap) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* kbuf = reinterpret_cast<bf16*>(smem_raw);
   bf16* vbuf = kbuf + DSTAGES * TILE_ELEMS;
@@ -724,7 +741,7 @@ __global__ void __launch_bounds__(THREADS, D <= 128 ? (DSTAGES == 2 ? 3 : 2) : 1
       }
       if (key_base + warp * 16 < total && (key_base + warp * 16 + 16 > lo || key_base + warp * 16 < keep_first))
         warp_tile<2>(st, qf, kbuf + stage * TILE_ELEMS, vbuf + stage * TILE_ELEMS, warp * 16, key_base, row_lo, row_hi, scale_log2, row_slope,
-                     keep_first);
+                     keep_first, cap);
       __syncthreads();
     }
     cp_async_wait<0>();
@@ -868,7 +885,7 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
                             int nkv, int page_size, int n_pages, int window, int chunk, float scale, float* scratch_o,
                             float* scratch_ml, int* counters, int max_pieces, int decode_blocks,
                             const FusedQK& fq, const float* sinks, const float* slopes, int keep_first, int out_head,
-                            cudaStream_t stream) {
+                            float softcap, cudaStream_t stream) {
   ATT_REQUIRE(out_head > 0 && out_head <= DV && out_head % 8 == 0,
               "attention: an output head has %d elements, in steps of 8 up to %d", out_head, DV);
   ATT_REQUIRE(!fq.qkv || (DV == D && out_head == D), "attention: the form that works from the projection has heads of one size");
@@ -879,7 +896,9 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
                   ((uintptr_t)out % 8) == 0,
               "attention: q and the pages must be 16-byte aligned, the output 8-byte aligned");
   const int G = nq / nkv;
-  const float scale_log2 = scale * LOG2E;
+  ATT_REQUIRE(softcap >= 0.f, "attention: a cap on the scores must be positive");
+  const NhvScoreCap cap = nhv_score_cap(scale, softcap);
+  const float scale_log2 = softcap > 0.f ? 1.0f : scale * LOG2E;
   static bool attr_set = false;
   static int sms = 0;
   if (!attr_set) {
@@ -912,12 +931,12 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
       if (wide)
         nhv_launch(attn_prefill_kernel<2>, grid, THREADS, prefill_smem_bytes<2>(), stream,
             (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv_pages, block_table, bt_stride, cu_q, kv_len,
-            n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first, out_head);
+            n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first, out_head, cap);
     }
     if (!wide)
       nhv_launch(attn_prefill_kernel<1>, grid, THREADS, prefill_smem_bytes<1>(), stream,
           (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv_pages, block_table, bt_stride, cu_q, kv_len,
-          n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first, out_head);
+          n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, tokens_per_block, sinks, slopes, keep_first, out_head, cap);
   }
   if (n_decode_seqs > 0) {
     ATT_REQUIRE(scratch_o && scratch_ml && counters && max_pieces > 0 && decode_blocks > 0,
@@ -934,7 +953,7 @@ static int attention_launch(const void* q, int q_stride, void* out, int out_stri
     decode_blocks = resident;
     nhv_launch(attn_decode_kernel, dim3(decode_blocks), THREADS, kDecodeSmemBytes, stream,
         (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv_pages, block_table, bt_stride, cu_q, kv_len,
-        scratch_o, scratch_ml, counters, n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, max_pieces, fq, sinks, slopes, keep_first, out_head);
+        scratch_o, scratch_ml, counters, n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale_log2, max_pieces, fq, sinks, slopes, keep_first, out_head, cap);
   }
   const cudaError_t e = cudaPeekAtLastError();
   if (e != cudaSuccess) {
@@ -950,11 +969,11 @@ NHV_API int NHV_FN(nhv_attn_mma_d)(const void* q, int q_stride, void* out, int o
                                    int nkv, int page_size, int n_pages, int window, int chunk, float scale, float* scratch_o,
                                    float* scratch_ml, int* counters, int max_pieces, int decode_blocks,
                                    const float* sinks, const float* slopes, int keep_first, int out_head,
-                                   cudaStream_t stream) {
+                                   float softcap, cudaStream_t stream) {
   FusedQK none = {};
   return attention_launch(q, q_stride, out, out_stride, kv_pages, block_table, bt_stride, cu_q, kv_len, n_seqs,
                           n_prefill_tokens, n_prefill_seqs, n_decode_seqs, nq, nkv, page_size, n_pages, window, chunk, scale,
-                          scratch_o, scratch_ml, counters, max_pieces, decode_blocks, none, sinks, slopes, keep_first, out_head, stream);
+                          scratch_o, scratch_ml, counters, max_pieces, decode_blocks, none, sinks, slopes, keep_first, out_head, softcap, stream);
 }
 
 // 1 if this head size has the form of the decode kernel that works from the projection's output.
@@ -991,5 +1010,5 @@ NHV_API int NHV_FN(nhv_attn_mma_decode_fused_d)(const void* qkv, int qkv_stride,
   fq.weight_offset = weight_offset;
   return attention_launch(qkv, qkv_stride, out, out_stride, kv_pages, block_table, bt_stride, cu_q, kv_len, n_seqs, 0, 0,
                           n_seqs, nq, nkv, page_size, n_pages, window, chunk, scale, scratch_o, scratch_ml, counters, max_pieces,
-                          1, fq, nullptr, nullptr, 0, D, stream);
+                          1, fq, nullptr, nullptr, 0, D, 0.f, stream);
 }

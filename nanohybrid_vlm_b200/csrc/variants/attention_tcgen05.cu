@@ -179,7 +179,8 @@ struct alignas(64) Params {
   int out_head;           // elements between two heads of the output, up to DV: that many are written
   int q_stride, out_stride, bt_stride, n_seqs, nq, nkv, page_size, n_pages, window, chunk, tokens_per_block;
   int keep_first;         // with a window: keys at positions below it stay visible (their tiles come first)
-  float scale_log2;
+  float scale_log2;       // 1 with capped scores, which are in log2 units already
+  NhvScoreCap cap;        // in == 0: none
 };
 
 __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tcgen05_kernel(const __grid_constant__ Params p) {
@@ -387,6 +388,15 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tc
       // and the scaling folded into the exponent's multiply-add.  A tile that some row of the block sees only
       // in part takes the masked path.
       const bool masked = !(key_base >= all_lo && key_base + BN - 1 <= all_hi);
+      if (p.cap.in != 0.f) {
+#pragma unroll
+        for (int i = 0; i < BN; i += 2) {
+          float a = __uint_as_float(sr[i >> 5][i & 31]), b = __uint_as_float(sr[i >> 5][(i & 31) + 1]);
+          nhv_cap_scores(a, b, p.cap);
+          sr[i >> 5][i & 31] = __float_as_uint(a);
+          sr[i >> 5][(i & 31) + 1] = __float_as_uint(b);
+        }
+      }
       if (p.slopes) {                                           // score - slope * (row - key), before maximum and mask
         const float at0 = slope * (float)(key_base - row_hi);
 #pragma unroll
@@ -551,7 +561,7 @@ NHV_API int NHV_FN(nhv_attn_tcgen05_d)(const void* q, int q_stride, void* out, i
                                        const int* block_table, int bt_stride, const int* cu_q, const int* kv_len,
                                        int n_seqs, int n_prefill_tokens, int n_prefill_seqs, int nq, int nkv,
                                        int page_size, int n_pages, int window, int chunk, float scale, const float* sinks,
-                                       const float* slopes, int keep_first, int out_head, cudaStream_t stream) {
+                                       const float* slopes, int keep_first, int out_head, float softcap, cudaStream_t stream) {
   ATT_REQUIRE(out_head > 0 && out_head <= DV && out_head % 8 == 0,
               "attention (tcgen05): an output head has %d elements, in steps of 8 up to %d", out_head, DV);
   ATT_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention: kept first keys go with a window");
@@ -601,7 +611,9 @@ NHV_API int NHV_FN(nhv_attn_tcgen05_d)(const void* q, int q_stride, void* out, i
   p.chunk = chunk;
   p.keep_first = keep_first;
   p.tokens_per_block = BM / G;
-  p.scale_log2 = scale * LOG2E;
+  ATT_REQUIRE(softcap >= 0.f && (softcap == 0.f || !slopes), "attention (tcgen05): a cap on the scores is positive and goes without a distance term");
+  p.cap = nhv_score_cap(scale, softcap);
+  p.scale_log2 = softcap > 0.f ? 1.0f : scale * LOG2E;
   const int max_tiles = n_prefill_tokens / p.tokens_per_block + n_prefill_seqs;
   ATT_REQUIRE(max_tiles <= 65535, "attention: %d tiles of new tokens are beyond the grid's reach", max_tiles);
   cudaError_t e = nhv_launch(attn_tcgen05_kernel, dim3(nkv, max_tiles), THREADS, SMEM_BYTES, stream, p);

@@ -40,7 +40,7 @@ def get(head_dim: int, v_dim: int | None = None):
         from ..csrc.build import ensure_variant
         lib = ctypes.CDLL(ensure_variant("attention_mma.cu", {"NHV_ATTN_D": head_dim, **({} if v_dim == head_dim else {"NHV_ATTN_DV": v_dim})}))
         fn = getattr(lib, f"nhv_attn_mma_d{head_dim}")
-        fn.argtypes = [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, I, P, P, I, I, P]
+        fn.argtypes = [P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, I, P, P, I, I, F, P]
         fn.restype = c_int
         err = getattr(lib, f"nhv_attn_mma_last_error_d{head_dim}")
         err.restype = ctypes.c_char_p

@@ -50,14 +50,14 @@ _SIGNATURES = {
     "nhv_add_row_bias": [I, P, P, I, I, P],
     "nhv_clamped_glu": [I, P, P, I, I, F, F, P],
     "nhv_mlstm_scan": [I, P, P, I, P, I, P, F, P, ctypes.c_long, P, P, P, I, I, I, I, I, I, P],
-    "nhv_moe_route": [P, P, P, I, P, I, I, I, I, I, I, I, P],
+    "nhv_moe_route": [P, P, P, I, P, I, I, I, I, I, I, I, I, F, P],
     "nhv_moe_align": [P, I, I, I, P, P, P, P],
     "nhv_moe_gemm_simt": [I, I, P, P, I, P, P, P, P, I, I, I, I, F, F, F, P, P],
     "nhv_moe_gemm_mma": [I, I, P, P, I, P, P, P, P, I, I, I, I, F, F, F, P, P],
     "nhv_moe_gather_rows": [P, P, P, I, I, I, P],
     "nhv_moe_gemm_tcgen05": [I, P, P, P, P, I, P, P, I, I, I, F, F, F, P, P],
     "nhv_moe_combine": [I, P, P, P, P, P, I, P, P, P, I, I, I, I, P],
-    "nhv_attention_simt_ex": [I, P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, I, I, P],
+    "nhv_attention_simt_ex": [I, P, I, P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, I, I, F, P],
     "nhv_causal_filter_add": [I, P, P, I, P, I, P, P, P, ctypes.c_long, P, P, P, I, I, I, I, P],
     "nhv_latent_rope_store": [I, P, I, P, I, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, I, P],
     "nhv_gemm_nt_simt_batched": [I, P, P, P, I, I, I, I, I, I, I, I, ctypes.c_long, ctypes.c_long, ctypes.c_long, P],
@@ -77,6 +77,11 @@ _SIGNATURES = {
     "nhv_decay_scan": [I, P, P, P, P, I, P, P, P, P, ctypes.c_long, P, P, P, I, I, I, I, I, I, I, P],
     "nhv_streams_rmsnorm": [I, P, P, P, I, P, P, P, P, P, P, I, I, I, F, P],
     "nhv_row_norm_store": [I, P, I, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, P, P],
+    "nhv_heads_store": [I, P, I, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, I, F, I, P, I, P, ctypes.c_long,
+                        P, P, P, I, I, P],
+    "nhv_map_difference": [I, P, I, P, I, P, F, F, I, I, I, P],
+    "nhv_sandwich_stream": [I, P, P, P, P, P, P, I, I, F, F, F, F, I, P],
+    "nhv_embed_rmsnorm": [I, P, P, P, P, I, I, I, F, F, P],
     "nhv_decay_lowrank": [I, P, P, I, P, P, I, I, I, P],
 }
 

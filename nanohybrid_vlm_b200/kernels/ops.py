@@ -157,6 +157,34 @@ def streams_rmsnorm(out, dst, src, weight, eps: float, y=None, mix=None, write=N
          _ptr(write), _ptr(read), weight.data_ptr(), _ptr(rows), n_rows, S, width, float(eps), stream_ptr())
 
 
+def sandwich_stream(out, stream, y, post_weight, pre_weight, post_eps: float, pre_eps: float, post_offset: float = 0.0,
+                    pre_offset: float = 0.0, rows=None, write_stream: bool = True) -> None:
+    """Norms around a float32 residual stream [T, width]: s = stream[src] + y[src] / rms(y[src]) * (post_weight + post_offset),
+    written back to the stream unless ``rows`` gathers, and out[r] = s / rms(s) * (pre_weight + pre_offset) rounded once to
+    the storage type; src = rows[r] or r.  All in 32-bit."""
+    _need_cuda(out, stream, y, post_weight, pre_weight, rows)
+    _contig("out", out); _contig("stream", stream); _contig("y", y)
+    width = stream.shape[-1]
+    assert stream.dtype == torch.float32 and y.shape == stream.shape and y.dtype == out.dtype
+    assert post_weight.numel() == pre_weight.numel() == width and post_weight.dtype == pre_weight.dtype == out.dtype
+    n_rows = rows.numel() if rows is not None else stream.numel() // width
+    assert out.numel() == n_rows * width and (rows is None or rows.dtype == torch.int32)
+    call("nhv_sandwich_stream", dtype_code(out), out.data_ptr(), stream.data_ptr(), y.data_ptr(), post_weight.data_ptr(),
+         pre_weight.data_ptr(), _ptr(rows), n_rows, width, float(post_eps), float(pre_eps), float(post_offset),
+         float(pre_offset), int(bool(write_stream and rows is None)), stream_ptr())
+
+
+def embed_rmsnorm(out, table, ids, weight, eps: float, weight_offset: float = 0.0) -> None:
+    """out [T, width] float32 = table[ids] / rms(table[ids]) * (weight + weight_offset): the looked-up rows through an RMS
+    norm, as the start of a residual stream kept in 32-bit."""
+    _need_cuda(out, table, ids, weight)
+    _contig("out", out); _contig("table", table)
+    assert ids.dtype == torch.int32 and out.dtype == torch.float32 and out.shape[1] == table.shape[1] == weight.numel()
+    assert weight.dtype == table.dtype
+    call("nhv_embed_rmsnorm", dtype_code(table), out.data_ptr(), table.data_ptr(), ids.data_ptr(), weight.data_ptr(),
+         ids.numel(), table.shape[1], table.shape[0], float(eps), float(weight_offset), stream_ptr())
+
+
 def scaled_sum(out, a, b, ca: float, cb: float) -> None:
     """out = ca * a + cb * b elementwise (sums in 32-bit)."""
     _need_cuda(out, a, b)
@@ -639,14 +667,15 @@ def mlstm_scan(y, proj, gates, gate_bias, cap: float, state, batch, H: int, d: i
 
 
 def moe_route(ids, weights, logits, correction, n_outputs: int, n_groups: int, keep: int, scores: str = "softmax",
-              renorm: bool = True) -> None:
+              renorm: bool = True, group_best: int = 1, factor: float = 1.0) -> None:
     """The router's choice per token.  logits [T, >= n_outputs] float32 (a view with unit column stride; further columns
     are not read), correction [n_outputs] float32 or None -> ids [T, top] int32 and weights [T, top] float32.
     Scores are the softmax over all outputs; the choice is by score + correction among the outputs of the ``keep`` best
     of ``n_groups`` groups of neighbours (a group's score: its largest choice score); the weights are the chosen scores
     divided by their sum (+ 1e-20).  ``scores`` "sigmoid": each output's score is the sigmoid of its logit;
     ``renorm`` False: the weights are the chosen scores as they are.  ``scores`` "chosen_softmax": the choice is by the
-    logit + correction (a bias), and the weights are the softmax of these over the chosen alone."""
+    logit + correction (a bias), and the weights are the softmax of these over the chosen alone.  ``group_best`` 2: a
+    group's score is the sum of its two largest choice scores.  ``factor`` multiplies the weights."""
     kinds = ("softmax", "sigmoid", "chosen_softmax")
     assert scores in kinds
     _need_cuda(ids, weights, logits, correction)
@@ -655,7 +684,7 @@ def moe_route(ids, weights, logits, correction, n_outputs: int, n_groups: int, k
     assert ids.is_contiguous() and weights.is_contiguous() and logits.stride(1) == 1 and logits.shape[0] == T
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == n_outputs)
     call("nhv_moe_route", ids.data_ptr(), weights.data_ptr(), logits.data_ptr(), logits.stride(0), _ptr(correction), T,
-         n_outputs, n_groups, keep, top, kinds.index(scores), int(bool(renorm)), stream_ptr())
+         n_outputs, n_groups, keep, top, kinds.index(scores), int(bool(renorm)), int(group_best), float(factor), stream_ptr())
 
 
 MOE_TILE_SIMT = 16      # rows of one expert that a block of the CUDA-core products takes (MG_BM of csrc/moe.cu)
@@ -868,14 +897,68 @@ def row_norm_store(qkv, q_out, q_head: int, kv_pages, slot_mapping, positions, c
          0 if v_first is None else v_first.stride(0), _ptr(v_share), stream_ptr())
 
 
+def heads_store(qkv, q_out, q_head: int, kv_pages, slot_mapping, batch, cos_sin, rotary_dim: int, nq: int, nkv: int, dk: int,
+                dv: int, eps: float | None, q_weight=None, k_weight=None, maps: int = 1, values_from_keys: bool = False,
+                taps=None, state=None, temperature=None) -> None:
+    """qkv [T, >= (nq + nkv) * maps * dk (+ nkv * dv)] -> queries q_out [T, nq * maps * q_head] and K / V rows in kv_pages
+    [pages, 2, nkv, page_size, row] at slot_mapping (None: queries only), for heads of ``maps`` independent query / key pairs
+    over one value head: map m of a query head goes to elements [m dk, (m + 1) dk) of its q_head, zeros elsewhere, map m
+    of a key head to the same elements of the head's row.
+    ``taps`` [K, (nq + nkv) * maps * dk] (one row per tap, the newest token's last): q and k first pass a causal filter over time
+    per channel; ``state`` [slots, (K - 1) * channels] float32 holds each request's last K - 1 inputs and is moved on.
+    ``values_from_keys``: the values are the key heads after the filter.  Then the norm per head and map (eps None: none)
+    with its weight [dk], the rotation of the first ``rotary_dim`` elements by halves, and for the queries the factor
+    1 + coef ln(floor((position + 1) / every) + 1), ``temperature`` = (coef, every) or None.  All in 32-bit, one rounding."""
+    _need_cuda(qkv, q_out, kv_pages, slot_mapping, cos_sin, q_weight, k_weight, taps, state)
+    T, C = qkv.shape[0], (nq + nkv) * maps * dk
+    assert qkv.dim() == 2 and qkv.stride(1) == 1 and q_out.dtype == qkv.dtype
+    assert q_out.shape == (T, nq * maps * q_head) and q_out.stride(1) == 1
+    for w in (q_weight, k_weight):
+        assert w is None or (w.dtype == qkv.dtype and w.is_contiguous() and w.numel() == dk and eps is not None)
+    if kv_pages is not None:
+        _contig("kv_pages", kv_pages)
+        n_pages, two, h, page_size, row = kv_pages.shape
+        assert two == 2 and h == nkv and row >= max(maps * dk, dv) and kv_pages.dtype == qkv.dtype
+        assert slot_mapping.dtype == torch.int32 and slot_mapping.numel() >= T
+        assert qkv.shape[1] >= C + (0 if values_from_keys else nkv * dv)
+    else:
+        n_pages, page_size, row = 0, 0, max(maps * dk, dv)
+        assert qkv.shape[1] >= nq * maps * dk and taps is None
+    K = 0
+    if taps is not None:
+        K = taps.shape[0]
+        assert taps.shape == (K, C) and taps.is_contiguous() and taps.dtype == qkv.dtype
+        assert K == 1 or (state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1)
+    if cos_sin is not None:
+        assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1] == rotary_dim
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    call("nhv_heads_store", dtype_code(qkv), qkv.data_ptr(), qkv.stride(0), q_out.data_ptr(), q_out.stride(0), int(q_head),
+         _ptr(kv_pages), _ptr(slot_mapping), batch.positions.data_ptr(), _ptr(cos_sin), int(rotary_dim),
+         0 if cos_sin is None else cos_sin.shape[0], T, nq, nkv, int(maps), dk, dv, row, page_size, n_pages,
+         -1.0 if eps is None else float(eps), _ptr(q_weight), _ptr(k_weight), int(bool(values_from_keys)), float(coef),
+         int(every), _ptr(taps), K, _ptr(state) if K > 1 else None, state.stride(0) if K > 1 else 0, batch.cu_q.data_ptr(),
+         batch.q_start.data_ptr(), batch.state_slots.data_ptr(), batch.n_seqs, int(batch.n_prefill_seqs > 0), stream_ptr())
+
+
+def map_difference(out, a, share, factor: float, eps: float, heads: int, dv: int) -> None:
+    """Two attention maps per head brought together: a [T, heads * 2 * dv] (head by head, map 1 then map 2), ``share`` [1]
+    float32: o = a1 - share * a2, out [T, heads * dv] = o / sqrt(mean(o^2) + eps) * factor, the mean over a head."""
+    _need_cuda(out, a, share)
+    T = out.shape[0]
+    assert a.dim() == out.dim() == 2 and a.stride(1) == out.stride(1) == 1 and a.dtype == out.dtype
+    assert out.shape == (T, heads * dv) and a.shape == (T, 2 * heads * dv) and share.dtype == torch.float32 and share.numel() == 1
+    call("nhv_map_difference", dtype_code(out), out.data_ptr(), out.stride(0), a.data_ptr(), a.stride(0), share.data_ptr(),
+         float(factor), float(eps), T, heads, dv, stream_ptr())
+
+
 def attention_sink_simt(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: int, n_tokens: int, nq: int, nkv: int,
                         dk: int, dv: int, scale: float, sinks=None, window: int = 0, chunk: int = 0, slopes=None,
-                        keep_first: int = 0) -> None:
+                        keep_first: int = 0, softcap: float | None = None) -> None:
     """Causal attention of this step's tokens over the pages with key heads of dk and value heads of dv elements:
     q [T, nq*dk] -> out [T, nq*dv].  ``sinks`` [nq] float32: a term exp(sink) in each head's softmax denominator.
     ``window`` > 0: the last ``window`` keys only; ``chunk`` > 0: only the keys of the query's own chunk of ``chunk``
     positions, counted from position 0 of the request.  ``slopes`` [nq] float32: head h's score loses slopes[h] times
-    the distance between query and key.  Pages with one plane ([pages, 1, nkv, page_size, row]): a row is the key and
+    the distance between query and key.  ``softcap``: scores become softcap * tanh(score / softcap).  Pages with one plane ([pages, 1, nkv, page_size, row]): a row is the key and
     its leading dv elements are the value."""
     _need_cuda(out, q, kv_pages, block_table, cu_q, kv_len, sinks, slopes)
     _contig("kv_pages", kv_pages)
@@ -888,14 +971,14 @@ def attention_sink_simt(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: int
     call("nhv_attention_simt_ex", dtype_code(q), q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0),
          kv_pages.data_ptr(), block_table.data_ptr(), block_table.stride(0), cu_q.data_ptr(), kv_len.data_ptr(),
          n_seqs, n_tokens, nq, nkv, dk, dv, row, page_size, n_pages, int(window), int(chunk), float(scale), _ptr(sinks),
-         _ptr(slopes), planes, int(keep_first), stream_ptr())
+         _ptr(slopes), planes, int(keep_first), float(softcap or 0.0), stream_ptr())
 
 
 SINK_ATTENTION_ON_TENSOR_CORES = True     # tests switch it off to compare with the CUDA-core kernel at the same shapes
 
 
 def attention_sink(out, q, kv_pages, tables, batch, nq: int, nkv: int, dk: int, dv: int, scale: float, sinks=None,
-                   window: int = 0, chunk: int = 0, slopes=None, keep_first: int = 0) -> None:
+                   window: int = 0, chunk: int = 0, slopes=None, keep_first: int = 0, softcap: float | None = None) -> None:
     """Attention of the step's tokens over the cache for layers with a sink and / or value heads of another size
     than their key heads: picks the kernel for the dtype and sizes.  bfloat16 with page rows and key heads of one size
     (in steps of 16) and value heads of at most that size (in steps of 8) runs on the tensor cores like ``attention``;
@@ -904,10 +987,10 @@ def attention_sink(out, q, kv_pages, tables, batch, nq: int, nkv: int, dk: int, 
             and kv_pages.shape[1] == 2 and attention_mma.supports(dk, nq, nkv, batch.n_seqs)):
         attention_tensor_core(out, q, kv_pages, tables.block_tables, batch.cu_q, batch.kv_len, batch.n_seqs,
                               batch.n_prefill_tokens, batch.n_prefill_seqs, batch.n_decode_seqs, batch.max_kv_len,
-                              nq, nkv, dk, scale, window, sinks, chunk, slopes, keep_first, dv)
+                              nq, nkv, dk, scale, window, sinks, chunk, slopes, keep_first, dv, softcap)
         return
     attention_sink_simt(out, q, kv_pages, tables.block_tables, batch.cu_q, batch.kv_len, batch.n_seqs, batch.n_tokens,
-                        nq, nkv, dk, dv, scale, sinks, window, chunk, slopes, keep_first)
+                        nq, nkv, dk, dv, scale, sinks, window, chunk, slopes, keep_first, softcap)
 
 
 def linear_f32(out, x, weight) -> None:
@@ -1017,7 +1100,7 @@ def _attention_decode_tma(out, q, qkv, kv_pages, block_table, batch_cu_q, batch_
                           head_dim: int, scale: float, window: int, q_weight=None, k_weight=None, cos_sin=None,
                           positions=None, slot_mapping=None, rotary_dim: int = 0, eps: float = 0.0,
                           weight_offset: float = 0.0, store: bool = False, sinks=None, chunk: int = 0,
-                          keep_first: int = 0, v_head: int | None = None) -> None:
+                          keep_first: int = 0, v_head: int | None = None, softcap: float | None = None) -> None:
     v_head = v_head or head_dim
     launch, blocks = attention_decode.get(head_dim, attention_mma.value_size(head_dim, v_head))
     n_pages, two, h, page_size, d = kv_pages.shape
@@ -1031,7 +1114,7 @@ def _attention_decode_tma(out, q, qkv, kv_pages, block_table, batch_cu_q, batch_
            batch_kv_len.data_ptr(), n_seqs, nq, nkv, page_size, n_pages, int(window), int(chunk), float(scale), part_o.data_ptr(),
            part_ml.data_ptr(), counters.data_ptr(), _ptr(q_weight), _ptr(k_weight), _ptr(cos_sin), _ptr(positions),
            _ptr(slot_mapping), int(rotary_dim), 0 if cos_sin is None else cos_sin.shape[0], 1 if store else 0, float(eps),
-           float(weight_offset), _ptr(sinks), int(keep_first), v_head, stream_ptr())
+           float(weight_offset), _ptr(sinks), int(keep_first), v_head, float(softcap or 0.0), stream_ptr())
 
 
 def attention_decode_fused(out, qkv, kv_pages, tables, batch, nq: int, nkv: int, head_dim: int, scale: float,
@@ -1092,7 +1175,7 @@ def attention_tcgen05_error(head_dim: int) -> int:
 def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: int, n_prefill_tokens: int,
                           n_prefill_seqs: int, n_decode_seqs: int, max_kv_len: int, nq: int, nkv: int, head_dim: int,
                           scale: float, window: int = 0, sinks=None, chunk: int = 0, slopes=None, keep_first: int = 0,
-                          v_head: int | None = None) -> None:
+                          v_head: int | None = None, softcap: float | None = None) -> None:
     """bfloat16 attention on the tensor cores.  Prompt portions go to the tcgen05 kernel, requests with
     one new token to the kernel that streams the cache with TMA, each where its shape is supported; what
     neither takes runs in the mma.sync kernel, whose single-token path shares a request's tiles between
@@ -1103,7 +1186,8 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
     ``keep_first`` > 0 (with a window): the keys at positions below it stay visible; in every kernel their tiles come
     before the window's.
     ``v_head`` (in steps of 8, up to ``head_dim``): the elements of a value head, where they are fewer: the leading ones
-    of a page's value row; out is then [T, nq * v_head]."""
+    of a page's value row; out is then [T, nq * v_head].
+    ``softcap``: scores become softcap * tanh(score / softcap) in 32-bit, before the distance term."""
     _need_cuda(out, q, kv_pages, block_table, cu_q, kv_len, sinks, slopes)
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == nq and sinks.is_contiguous())
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == nq and slopes.is_contiguous())
@@ -1115,7 +1199,7 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
     v_head = v_head or head_dim
     v_dim = attention_mma.value_size(head_dim, v_head)
     launch, tile = attention_mma.get(head_dim, v_dim)[:2]
-    if (n_prefill_tokens > 0 and USE_TCGEN05_ATTENTION and (slopes is None or scale > 0)
+    if (n_prefill_tokens > 0 and USE_TCGEN05_ATTENTION and (slopes is None or (scale > 0 and not softcap))
             and attention_tcgen05.supports(head_dim, nq, nkv, page_size)):
         # prompt portions on the 5th-generation tensor cores; single tokens stay with the split kernel below
         library.LAUNCHES += 1
@@ -1123,7 +1207,7 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
             q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), kv_pages.data_ptr(), block_table.data_ptr(),
             block_table.stride(0), cu_q.data_ptr(), kv_len.data_ptr(), n_seqs, n_prefill_tokens, n_prefill_seqs,
             nq, nkv, page_size, n_pages, int(window), int(chunk), float(scale), _ptr(sinks), _ptr(slopes), int(keep_first),
-            v_head, stream_ptr())
+            v_head, float(softcap or 0.0), stream_ptr())
         if n_decode_seqs == 0:
             return
         n_prefill_tokens = n_prefill_seqs = 0
@@ -1132,7 +1216,7 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
         # single tokens: the kernel that streams the cache with TMA; what is left for the launch below are the
         # prompt portions (if the tcgen05 kernel did not take them)
         _attention_decode_tma(out, q, None, kv_pages, block_table, cu_q, kv_len, n_seqs, nq, nkv, head_dim, scale, window,
-                              sinks=sinks, chunk=chunk, keep_first=keep_first, v_head=v_head)
+                              sinks=sinks, chunk=chunk, keep_first=keep_first, v_head=v_head, softcap=softcap)
         if n_prefill_tokens == 0:
             return
         n_decode_seqs = 0
@@ -1152,7 +1236,8 @@ def attention_tensor_core(out, q, kv_pages, block_table, cu_q, kv_len, n_seqs: i
     launch(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), kv_pages.data_ptr(), block_table.data_ptr(),
            block_table.stride(0), cu_q.data_ptr(), kv_len.data_ptr(), n_seqs, n_prefill_tokens, n_prefill_seqs,
            n_decode_seqs, nq, nkv, page_size, n_pages, int(window), int(chunk), float(scale), _ptr(scratch_o), _ptr(scratch_ml),
-           _ptr(counters), max_pieces, blocks, _ptr(sinks), _ptr(slopes), int(keep_first), v_head, stream_ptr())
+           _ptr(counters), max_pieces, blocks, _ptr(sinks), _ptr(slopes), int(keep_first), v_head, float(softcap or 0.0),
+           stream_ptr())
 
 
 _sm_counts: dict = {}

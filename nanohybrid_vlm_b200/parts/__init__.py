@@ -1,4 +1,4 @@
-from . import (attention, block, delta_rule, embedding, feed_forward, input_filter, latent_attention, linear_recurrence, mlstm, moe, norm,  # noqa: F401
+from . import (attention, block, delta_rule, differential_attention, embedding, feed_forward, input_filter, latent_attention, linear_recurrence, mlstm, moe, norm,  # noqa: F401
                parallel_mixer, position, sink_attention, state_space)    # (importing registers the built-in parts)
 from .base import (BLOCKS, CONNECTIONS, EMBEDDINGS, FEED_FORWARDS, FILTERS, HEADS, MIXERS, NORMS, POSITIONS, Block, InputFilter, SharedPagesNeed, StreamConnection, BuildEnv, CacheView, CompositeNeed,
                    Embedding,

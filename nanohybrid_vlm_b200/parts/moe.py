@@ -19,7 +19,8 @@ chosen expert's output is multiplied by its weight; "input": its input is, out =
 are the softmax of these over the chosen alone), ``correction_source`` (the checkpoint's name of the correction, default
 "correction"), ``unit`` ("glu", the default, or "relu2": experts without a gate, down(relu(up x)^2), and no ``gate``
 tensors) and ``up_shift`` (what is added to the up half, 1 unless given): limit None, alpha 1, up_shift 0 make the
-experts plain gated units, down(silu(gate x) * (up x)).
+experts plain gated units, down(silu(gate x) * (up x)); ``group_best`` (1, the default, or 2: a group's score is the sum of its
+two largest choice scores) and ``weight_factor`` (a factor on the weights, 1 unless given).
 
 Router: z = router(x) with 32-bit sums; s = softmax(z) over all outputs; choice by s + correction; the weights of the
 chosen are their s divided by the sum of the chosen s (+ 1e-20).  The output is the weighted sum of the chosen experts'
@@ -89,6 +90,8 @@ class RoutedMoE(FeedForward):
         self.up_shift = float(spec.get("up_shift", 1.0))
         self.scores = spec.get("scores", "softmax")
         self.renorm = bool(spec.get("renorm", True))
+        self.group_best = int(spec.get("group_best", 1))
+        self.weight_factor = float(spec.get("weight_factor", 1.0))
         self.weight_on = spec.get("weight_on", "output")
         self.unit = spec.get("unit", "glu")
         self.correction_source = spec.get("correction_source", "correction")
@@ -153,7 +156,7 @@ class RoutedMoE(FeedForward):
         ids = self.new(T, self.top, dtype=torch.int32)
         weights = self.new(T, self.top, dtype=torch.float32)
         ops.moe_route(ids, weights, logits, self.w_correction if self.has_correction else None, self.N, self.groups, self.keep,
-                      scores=self.scores, renorm=self.renorm)
+                      scores=self.scores, renorm=self.renorm, group_best=self.group_best, factor=self.weight_factor)
         on_input = self.weight_on == "input"
         # a weight on an expert's input is a factor on the 32-bit sums of its two first products
         y, slot_pos = ops.moe_experts(x, self.w_gate if self.unit == "glu" else None, self.w_up, self.w_down, ids, self.limit, self.alpha, self.up_shift,

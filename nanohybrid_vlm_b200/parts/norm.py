@@ -12,7 +12,8 @@ Over a residual stream of several copies (``forward_streams``, and ``forward_add
 connection) one kernel rebuilds the copies from the pending output, sums what the next sub-block reads and norms it.
 
 Over a residual stream kept in float32 (``forward_add`` / ``forward_add_rows`` given a :class:`Pending`) the terms
-are added in 32-bit, the statistics and the product with the weight are 32-bit, and the result is rounded once.
+are added in 32-bit, the statistics and the product with the weight are 32-bit, and the result is rounded once.  A term
+that still has to pass an RMS norm of its own (``Pending.post``) is normed, added and the sum normed in one kernel.
 """
 from __future__ import annotations
 
@@ -90,10 +91,32 @@ class RMSNorm(Norm):
         ops.rmsnorm(out, x, self.w_weight, self.eps, weight_offset=self.weight_offset)
         return out
 
+    def forward_embedding(self, table, token_ids):
+        """The looked-up rows of ``table`` through this norm, as a float32 stream [T, width]."""
+        self._plain_only()
+        out = self.new(token_ids.numel(), self.width, dtype=torch.float32)
+        ops.embed_rmsnorm(out, table, token_ids, self.w_weight, self.eps, self.weight_offset)
+        return out
+
+    def _sandwich(self, x, residual, rows):
+        """The pending output through its own RMS norm onto the stream, and this norm of the sum, in one kernel; None where
+        the two norms do not allow it."""
+        post = x.post
+        if (not isinstance(post, RMSNorm) or len(x.terms) != 1 or x.terms[0][1] != 1.0 or self.groups != 1 or post.groups != 1
+                or post.post_scale is not None):
+            return None
+        out = self.new(residual.shape[0] if rows is None else rows.numel(), self.width)
+        ops.sandwich_stream(out, residual, x.terms[0][0], post.w_weight, self.w_weight, post.eps, self.eps, post.weight_offset,
+                            self.weight_offset, rows=rows)
+        return out
+
     def forward_add(self, x, residual):
         if isinstance(x, Pending):
             if self.post_scale is not None:
                 self._plain_only()
+            fused = self._sandwich(x, residual, None)
+            if fused is not None:
+                return fused
             x = x.settled()
             out = self.new(*residual.shape)
             ops.rmsnorm_stream(out, residual, self.w_weight, self.eps, addends=x.terms, weight_offset=self.weight_offset,
@@ -108,6 +131,9 @@ class RMSNorm(Norm):
         if isinstance(x, Pending) and x.connection is not None:      # the norm of the sum of the new copies
             return self._streams(x, residual, x.connection.streams, None, None, rows)
         if isinstance(x, Pending):
+            fused = self._sandwich(x, residual, rows)
+            if fused is not None:
+                return fused
             x = x.settled()
             out = self.new(rows.numel(), residual.shape[-1])
             ops.rmsnorm_stream(out, residual, self.w_weight, self.eps, addends=x.terms, rows=rows, write_stream=False,

@@ -27,7 +27,11 @@ biases on q and k only, ``qk_norm_scope`` ("head", the default, or "projection":
 mean square over the whole query projection, the key heads likewise, and the weights ``q.norm`` / ``k.norm`` have that
 size; before the rotation, with a weight), ``value_mix`` (None; "source": the layer leaves its values to the later layers
 of the step; "mixed": the values become (1 - lambda) v + lambda v_source of the same token, lambda a learned number
-``vmix``, and the mixed values are what the pages keep; with ``qk_norm_scope`` "projection" only).
+``vmix``, and the mixed values are what the pages keep; with ``qk_norm_scope`` "projection" only), ``conv_taps`` (K: q and k
+pass a causal filter of K taps over time per channel, ``q.conv`` / ``k.conv`` [channels, K], directly after the projection; values
+that are the keys are the filtered ones; the last K - 1 projected q and k of each request are kept beside the pages),
+``query_temperature`` (None, or (coef, every): the queries are multiplied by 1 + coef ln(floor((position + 1) / every) + 1)
+after norm and rotation).
 
 Tensors: ``qkv`` [(nq + nkv) d (+ nkv dv) (+ nq dv), width], rows q then k then v then g, packed from the
 checkpoint's ``q``, ``k``, ``v``, ``g`` (those that exist); ``qk_bias`` [(nq + nkv) d] from ``q.b``, ``k.b``; ``sink``
@@ -38,7 +42,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import MIXERS, Mixer, PagedKVNeed
+from .base import MIXERS, CompositeNeed, FixedStateNeed, Mixer, PagedKVNeed
 from .spec import ParamDecl, Source
 
 
@@ -105,6 +109,21 @@ class SinkAttention(Mixer):
                              "and values of the layer's own, without biases")
         if self.value_mix and not self.rows:
             raise ValueError("mixed values are offered with a norm over the whole projection")
+        self.taps = int(spec.get("conv_taps") or 0)
+        self.temperature = spec.get("query_temperature")
+        if self.temperature is not None:
+            coef, every = self.temperature
+            self.temperature = (float(coef), int(every))
+            if self.temperature[1] < 1:
+                raise ValueError("a query temperature changes every so many positions, at least one")
+        if self.taps < 0:
+            raise ValueError("a filter over time has at least one tap")
+        # heads that pass a filter or a temperature go through a kernel of their own
+        self.prepared = self.taps > 0 or self.temperature is not None
+        if self.prepared and (self.rows or self.bias or not self.own_kv or self.rope_layout != "half"
+                              or (self.position is not None and self.eps is not None and self.norm_order != "before_rotation")):
+            raise ValueError("a filter over time or a query temperature goes with keys of the layer's own, without biases, normed "
+                             "per head before a rotation by halves")
         # what a page row and a query head hold: on the tensor cores keys and values of unequal size are padded to one
         self.D = self.d
         if self.rows and env.dtype == torch.bfloat16 and (self.dv > self.d or self.d % 16):
@@ -133,6 +152,9 @@ class SinkAttention(Mixer):
             decls.append(ParamDecl("q.norm", (self.q_size if self.rows else self.d,), init="norm"))
             if self.own_kv:
                 decls.append(ParamDecl("k.norm", (self.k_size if self.rows else self.d,), init="norm"))
+        if self.taps:
+            decls.append(ParamDecl("qk_conv", (self.q_size + self.k_size, self.taps), init="filter_taps",
+                                   sources=(Source("q.conv", 0, self.q_size), Source("k.conv", self.q_size, self.k_size))))
         if self.value_mix == "mixed":
             decls.append(ParamDecl("vmix", (1,), init="mix_share", storage="float32", sources=(Source("vmix", 0, 1, squeeze=True),)))
         if self.bias:
@@ -144,15 +166,27 @@ class SinkAttention(Mixer):
                 decls.append(ParamDecl("o.b", (H,), init="zeros_noise"))
         return decls
 
+    def bind(self, tensors):
+        super().bind(tensors)
+        if self.taps:
+            self.w_taps = self.w_qk_conv.t().contiguous()       # one row per tap: what the kernel reads side by side
+
     def cache_need(self):
-        return PagedKVNeed(self.nkv, self.D, self.keep_window, v_head_dim=self.dv, chunk=self.chunk,
-                           keep_first=self.keep_first)
+        pages = PagedKVNeed(self.nkv, self.D, self.keep_window, v_head_dim=self.dv, chunk=self.chunk,
+                            keep_first=self.keep_first)
+        if self.taps < 2:
+            return pages
+        return CompositeNeed((pages, FixedStateNeed(((self.taps - 1) * (self.q_size + self.k_size),))))
 
     def streamed_weights(self):
         return [(self.w_qkv, 0), (self.w_o, 0)]
 
     def forward(self, x, batch, cache):
         T = x.shape[0]
+        state = None
+        if self.taps > 1:
+            cache, kept = cache.children
+            state = kept.state
         qkv = self.new(T, self.q_size + self.k_size + self.v_size + self.g_size)
         ops.linear(qkv, x, self.w_qkv)
         rot = self.position.rotary() if self.position is not None else None
@@ -160,7 +194,12 @@ class SinkAttention(Mixer):
         q = self.new(T, self.nq * self.D)
         if cache.writes != self.own_kv:
             raise ValueError("a layer with keys of its own writes its pages; one without reads another run's (cache_from)")
-        if self.rows:
+        if self.prepared:
+            ops.heads_store(qkv, q, self.D, cache.pages, cache.tables.slot_mapping, batch, table, rotary_dim, self.nq, self.nkv,
+                            self.d, self.dv, self.eps, self.w_q_norm if self.norm_weight else None,
+                            self.w_k_norm if self.norm_weight else None, values_from_keys=self.values == "keys",
+                            taps=self.w_taps if self.taps else None, state=state, temperature=self.temperature)
+        elif self.rows:
             self._store_rows(qkv, q, batch, cache, table, rotary_dim)
         else:
             ops.rope_norm_store(qkv, q, cache.pages if cache.writes else None, cache.tables.slot_mapping, batch.positions,

@@ -41,6 +41,7 @@ INITS = {
     "filter_taps": _normal(0.3),                # short filters over time: large enough to show in the output
     "unit": _normal(1.0),
     "layer_scale": _normal(0.1, 0.5),
+    "map_share": _normal(0.1),                  # vectors whose inner products make a share near its constant
     "mix_share": _normal(0.2, 0.5),             # how much of the token before, or of another layer's values, enters a mix
     # how several copies of a residual stream are rebuilt from one another: near the identity
     "stream_mix": lambda shape, gen, device: torch.eye(shape[-1], device=device) * 0.8 + 0.1 * torch.empty(
