@@ -7,6 +7,7 @@
     python bench.py --designs nomudra        Nomudra beside a Muvonex of equal active size, the same way
     python bench.py --designs ginodra        Ginodra beside a Muvonex of equal size, the same way
     python bench.py --designs beputar        Beputar beside a Nomudra of the same width and expert sizes, the same way
+    python bench.py --designs kilisun        Kilisun beside a Nomudra and a Beputar of the same width and expert sizes
     python bench.py --designs vozorax        Vozorax beside a Ginodra of equal active size and a Nomudra, the same way
 
 The default run has the layer sizes of the Qwen3-8B-shaped configuration (36 layers, width 4096,
@@ -741,6 +742,26 @@ def vozorax_config(width: int, heads: int, ff: int, layers: int) -> dict:
                 layers=[dict((latent, window)[i % 2], mlp=dict(kind="dense", ff=ff) if i % 4 == 0 else moe) for i in range(layers)])
 
 
+def kilisun_config(width: int, heads: int, ff: int, layers: int) -> dict:
+    """In turn: differential attention in a window of 1,024 (two maps of 64 per head over values of 128, a quarter as many
+    key heads, capped scores), attention over all keys (heads of 128, three filter taps, values that are the keys), a
+    second differential layer that reads the first one's keys, and attention over all keys again.  The first layer of
+    every four has the dense feed-forward ``ff``; the others a mixture of 16 experts in 4 groups of which 2 are kept, a
+    token uses 4, and a shared expert: together as wide as ``ff`` (4 * 2/11 + 3/11 of it)."""
+    moe = dict(kind="moe", router=dict(experts=16, top=4, groups=dict(count=4, keep=2), scale=2.0),
+               expert=dict(ff=ff * 2 // 11, limit=7.0), shared=dict(ff=ff * 3 // 11, limit=7.0))
+    kv = max(heads // 4, 1)
+    maps = dict(heads=heads, kv_heads=kv, dim=64, vdim=128, scale=64 ** -0.5, diff=0.6, softcap=30.0,
+                rot=dict(base=500000.0, dims=64), mask=dict(size=1024))
+    full = dict(heads=heads, kv_heads=kv, dim=128, vdim=128, scale=128 ** -0.5, conv=3, q_temp=dict(coef=0.3, every=1024))
+    out = []
+    for i in range(layers):
+        mixer = full if i % 2 else (dict(maps, kv_from=i - 2) if i % 4 == 2 else maps)
+        out.append(dict(type="attention" if i % 2 else "attention_2", mixer=mixer,
+                        mlp=dict(kind="dense", ff=ff, limit=7.0) if i % 4 == 0 else moe))
+    return dict(architecture="Kilisun", vocab=DESIGN_VOCAB, width=width, norm=dict(eps=1e-6), layers=out, dtype="bfloat16")
+
+
 def qwen3_config_of_equal_size(width: int, heads: int, layers: int, layer_weights: float) -> dict:
     """A Qwen3 of this width whose layers hold as many weights as ``layer_weights`` (the feed-forward takes up the
     difference, rounded to 256)."""
@@ -756,8 +777,8 @@ def bench_designs(args) -> dict:
     Muvonex whose layers hold as many weights as a Nomudra token uses (``--designs nomudra``), or of Ginodra beside a
     Muvonex of equal size (``--designs ginodra``), or of Beputar beside a Nomudra of the same width and expert sizes
     (``--designs beputar``), or of Vozorax beside a Ginodra whose layers hold as many weights as a Vozorax token uses and
-    beside a Nomudra of the same width (``--designs vozorax``), and the time of each kind
-    of kernel in a prefill step (CUDA events around every launch of an eager run) with its share of the measured
+    beside a Nomudra of the same width (``--designs vozorax``), or of Kilisun beside a Nomudra and a Beputar of the same
+    width and expert sizes (``--designs kilisun``), and the time of each kind of kernel in a prefill step (CUDA events around every launch of an eager run) with its share of the measured
     roofline."""
     import torch
 
@@ -780,7 +801,8 @@ def bench_designs(args) -> dict:
              "latent_attention": "attention", "latent_expand": "attention", "general_delta": "delta_rule", "sigmoid_mul_heads": "act_mul",
              "relu_squared": "act_mul", "scale_softcap": "act_mul", "gelu_tanh": "act_mul", "postnorm_stream": "norm",
              "stream_round": "norm", "token_shift_mix": "token_shift", "decay_scan": "decay_scan", "decay_lowrank": "decay_prep",
-             "streams_rmsnorm": "norm", "row_norm_store": "rope_store"}
+             "streams_rmsnorm": "norm", "row_norm_store": "rope_store", "sandwich_stream": "norm", "embed_rmsnorm": "embed",
+             "heads_store": "rope_store", "map_difference": "maps"}
     kinds = {k: v for k, v in kinds.items() if hasattr(ops, k)}
     stock = {name: getattr(ops, name) for name in kinds}
     gen = torch.Generator().manual_seed(SEED)
@@ -967,6 +989,12 @@ def bench_designs(args) -> dict:
             results[name] = {"beputar": run_one(beputar_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB),
                              "nomudra": run_one(nomudra_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB)}
             continue
+        if args.designs == "kilisun":
+            # the same width, heads, expert count and expert sizes: all report the weights that a token uses
+            results[name] = {"kilisun": run_one(kilisun_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB),
+                             "nomudra": run_one(nomudra_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB),
+                             "beputar": run_one(beputar_config(sz["width"], sz["heads"], sz["ff"], layers), DESIGN_VOCAB)}
+            continue
         mcfg = muvonex_config(sz["width"], sz["heads"], sz["ff"], layers)
         m = run_one(mcfg, DESIGN_VOCAB)
         layer_weights = (m["weights_m"] * 1e6 - DESIGN_VOCAB * sz["width"]) / layers
@@ -998,7 +1026,7 @@ def main() -> int:
     ap.add_argument("--requests", type=int, default=0, help="fewer requests than the workload names (trying it out)")
     ap.add_argument("--breakdown", action="store_true",
                     help="time by kind of kernel in an eager run with --layers layers (default 2); prints one JSON line")
-    ap.add_argument("--designs", nargs="?", const="muvonex", default=None, choices=["muvonex", "nomudra", "ginodra", "beputar", "vozorax"],
+    ap.add_argument("--designs", nargs="?", const="muvonex", default=None, choices=["muvonex", "nomudra", "ginodra", "beputar", "vozorax", "kilisun"],
                     help="two designs side by side, prefill and decode throughput at a few layer sizes, one JSON line: "
                          "Muvonex beside a Qwen3 of equal size (the default), or Nomudra beside a Muvonex of equal active size")
     ap.add_argument("--design-size", default="all", choices=["all", *DESIGN_SIZES], help="one size of --designs")
