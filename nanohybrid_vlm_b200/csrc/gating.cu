@@ -137,14 +137,23 @@ NHV_API int nhv_clamped_glu(int dtype, void* out, const void* gate_up, int n_row
 // out[t, c] = x[t, c] * sigmoid(g[t, c / group]): one gate per head of `group` columns.  out may be x itself.
 // x_head: the distance between two heads in a row of x (group where the heads are packed; more where each head is
 // padded, as the output of attention over padded heads is).
-template <typename T>
+template <typename T, int VEC>
 __global__ void sigmoid_mul_heads_kernel(T* out, int out_stride, const T* x, int x_stride, const T* __restrict__ g,
                                          int g_stride, int width, int group, int x_head, size_t total) {
   pdl_prologue();
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+  for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC; i < total; i += (size_t)gridDim.x * blockDim.x * VEC) {
     const size_t t = i / width;
     const int c = (int)(i - t * width);
     const int h = c / group;
+    if constexpr (VEC == 8) {                                   // eight columns of one head
+      float v[8];
+      nhv_load8(v, x + t * x_stride + (size_t)h * x_head + (c - h * group));
+      const float s = sigmoid_f(to_f32<T>(g[t * g_stride + h]));
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= s;
+      nhv_store8(out + t * out_stride + c, v);
+      continue;
+    }
     out[t * out_stride + c] = from_f32<T>(to_f32<T>(x[t * x_stride + (size_t)h * x_head + (c - h * group)]) *
                                           sigmoid_f(to_f32<T>(g[t * g_stride + h])));
   }
@@ -156,12 +165,13 @@ NHV_API int nhv_sigmoid_mul_heads(int dtype, void* out, int out_stride, const vo
   NHV_REQUIRE(n_rows > 0 && width > 0 && group > 0 && width % group == 0 && x_head >= group,
               "sigmoid_mul_heads: %d columns do not divide into heads of %d", width, group);
   const size_t total = (size_t)n_rows * width;
-  if (dtype == NHV_F32)
-    nhv_launch(sigmoid_mul_heads_kernel<float>, gating_blocks(total), 256, 0, stream, (float*)out, out_stride, (const float*)x,
-               x_stride, (const float*)g, g_stride, width, group, x_head, total);
-  else if (dtype == NHV_BF16)
-    nhv_launch(sigmoid_mul_heads_kernel<__nv_bfloat16>, gating_blocks(total), 256, 0, stream, (__nv_bfloat16*)out, out_stride,
-               (const __nv_bfloat16*)x, x_stride, (const __nv_bfloat16*)g, g_stride, width, group, x_head, total);
+  const bool vec = group % 8 == 0 && x_head % 8 == 0 && out_stride % 8 == 0 && x_stride % 8 == 0 && aligned16(out) && aligned16(x);
+#define GO(T, V)                                                                                                        \
+  nhv_launch(sigmoid_mul_heads_kernel<T, V>, gating_blocks(total / V), 256, 0, stream, (T*)out, out_stride, (const T*)x, \
+             x_stride, (const T*)g, g_stride, width, group, x_head, total)
+  if (dtype == NHV_F32) { if (vec) GO(float, 8); else GO(float, 1); }
+  else if (dtype == NHV_BF16) { if (vec) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
+#undef GO
   else
     NHV_REQUIRE(false, "sigmoid_mul_heads: unknown dtype %d", dtype);
   NHV_CHECK_LAUNCH("sigmoid_mul_heads");

@@ -27,6 +27,8 @@
 #include "nhv_vec8.cuh"
 
 constexpr int HS_THREADS = 256;
+constexpr int HS_TOKENS = 4;             // the most tokens of a block
+constexpr int HS_TAPS = 4;               // filters of up to so many taps keep theirs in registers
 constexpr int HS_WARPS = 4;              // of the general kernel
 
 template <typename T>
@@ -42,71 +44,88 @@ struct HeadsStore {
   const float* cos_sin;
   long state_stride;
   int qkv_stride, q_out_stride, q_head, rotary_dim, max_position, n_tokens, n_seqs, nq, nkv, maps, dk, dv, row, page_size,
-      n_pages, K, v_from_k, units, temp_every;
+      n_pages, K, v_from_k, units, temp_every, one_each;
   float eps, temp_coef;
 };
 
-// What a unit (token, head and map) is and where its results go.
+// What a unit (head and map of a token) is and where its results go.
 template <typename T>
 struct HeadsUnit {
-  int t, kind, map, pos;                 // kind: 0 query, 1 key, 2 value
+  int kind, map;                         // kind: 0 query, 1 key, 2 value
   int col;                               // its first column of qkv
   T* dst;                                // its padded query head, or its row of the cache (null: not stored)
   T* dst_v;                              // v_from_k: the value row
 };
 
+// A token's facts, the same for all its units.
+struct HeadsToken {
+  int pos;
+  long row;                              // element offset of the token's K row of head 0 in the pages, or -1
+  // for the filter: how many tokens of this portion lie before it, whether the portion is this token alone, and its
+  // request's state (null: no slot; has_past: it holds inputs)
+  int before, single, has_past;
+  float* state;
+};
+
 template <typename T>
-__device__ __forceinline__ HeadsUnit<T> heads_unit(const HeadsStore<T>& p, long item) {
+__device__ __forceinline__ HeadsToken heads_token(const HeadsStore<T>& p, int t) {
+  HeadsToken k;
+  k.pos = p.positions ? p.positions[t] : 0;
+  k.row = -1;
+  if (p.kv_pages) {
+    const int slot = p.slot_mapping[t];
+    if (slot >= 0 && slot < p.n_pages * p.page_size) {
+      const int page = slot / p.page_size, off = slot - page * p.page_size;
+      k.row = ((long)page * 2 * p.nkv * p.page_size + off) * p.row;
+    }
+  }
+  k.before = k.single = k.has_past = 0;
+  k.state = nullptr;
+  if (p.taps) {
+    int lo = t;                                             // a step of single tokens: one request each
+    if (!p.one_each) {
+      lo = 0;
+      int hi = p.n_seqs - 1;
+      while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (p.cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+      }
+    }
+    const int first = p.cu_q[lo], slot = p.slots[lo];
+    k.before = t - first;
+    k.single = p.cu_q[lo + 1] - first == 1;
+    k.has_past = slot >= 0 && p.q_start[lo] > 0;
+    if (slot >= 0) k.state = p.state + (size_t)slot * p.state_stride;
+  }
+  return k;
+}
+
+template <typename T>
+__device__ __forceinline__ HeadsUnit<T> heads_unit(const HeadsStore<T>& p, int t, const HeadsToken& k, int x) {
   HeadsUnit<T> u;
-  u.t = (int)(item / p.units);
-  const int x = (int)(item - (long)u.t * p.units);
   const int nqm = p.nq * p.maps, nkm = p.nkv * p.maps;
+  auto head_of = [&](int i) { return p.maps == 1 ? i : p.maps == 2 ? i >> 1 : i / p.maps; };
   u.dst_v = nullptr;
-  u.pos = p.positions ? p.positions[u.t] : 0;
   if (x < nqm) {
     u.kind = 0;
-    u.map = x % p.maps;
+    u.map = x - head_of(x) * p.maps;
     u.col = x * p.dk;
-    u.dst = p.q_out + (size_t)u.t * p.q_out_stride + (size_t)x * p.q_head;
+    u.dst = p.q_out + (size_t)t * p.q_out_stride + (size_t)x * p.q_head;
     return u;
   }
   const int y = x - nqm;
   u.kind = y < nkm ? 1 : 2;
-  u.map = u.kind == 1 ? y % p.maps : 0;
-  const int g = u.kind == 1 ? y / p.maps : y - nkm;
+  const int g = u.kind == 1 ? head_of(y) : y - nkm;
+  u.map = u.kind == 1 ? y - g * p.maps : 0;
   u.col = u.kind == 1 ? x * p.dk : (nqm + nkm) * p.dk + g * p.dv;
-  const int slot = p.slot_mapping[u.t];
   u.dst = nullptr;
-  if (slot >= 0 && slot < p.n_pages * p.page_size) {
-    const int page = slot / p.page_size, off = slot - page * p.page_size;
+  if (k.row >= 0) {
     const size_t plane = (size_t)p.nkv * p.page_size * p.row;
-    T* k_row = p.kv_pages + (((size_t)page * 2 * p.nkv + g) * p.page_size + off) * p.row;
+    T* k_row = p.kv_pages + k.row + (size_t)g * p.page_size * p.row;
     u.dst = u.kind == 1 ? k_row : k_row + plane;
     if (p.v_from_k) u.dst_v = k_row + plane;
   }
   return u;
-}
-
-// The request of token t, for the filter: how many tokens of this portion lie before t, and the request's state.
-struct HeadsPast {
-  int before, single;
-  bool has_past;
-  float* state;                          // null: no slot
-};
-template <typename T>
-__device__ __forceinline__ HeadsPast heads_past(const HeadsStore<T>& p, int t) {
-  int lo = 0, hi = p.n_seqs - 1;
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (p.cu_q[mid] <= t) lo = mid; else hi = mid - 1;
-  }
-  HeadsPast h;
-  const int first = p.cu_q[lo], slot = p.slots[lo];
-  h.before = t - first;
-  h.single = p.cu_q[lo + 1] - first == 1;
-  h.has_past = slot >= 0 && p.q_start[lo] > 0;
-  h.state = slot >= 0 ? p.state + (size_t)slot * p.state_stride : nullptr;
-  return h;
 }
 
 template <typename T>
@@ -121,111 +140,150 @@ __device__ __forceinline__ const float* heads_angles(const HeadsStore<T>& p, int
   return p.cos_sin + (size_t)pos * p.rotary_dim;
 }
 
-// L lanes per unit, eight consecutive elements a lane: sizes in steps of 8, halves of the rotation too.
-template <typename T, int L>
-__global__ void __launch_bounds__(HS_THREADS) heads_store_vec_kernel(const HeadsStore<T> p) {
+// L lanes per unit, eight consecutive elements a lane: sizes in steps of 8, halves of the rotation too.  A block takes
+// `tokens` neighbouring tokens (gridDim.x) and all their units, or a share of them (gridDim.y); a unit's filter taps are read
+// once for its tokens.  TAPS: taps held in registers (0: no filter; filters of more taps read theirs per token, TAPS -1).
+template <typename T, int L, int TAPS>
+__global__ void __launch_bounds__(HS_THREADS) heads_store_vec_kernel(const HeadsStore<T> p, int tokens) {
+  __shared__ HeadsToken facts[HS_TOKENS];
+  __shared__ float temp[HS_TOKENS];
   pdl_prologue();
-  const long item = (long)blockIdx.x * (HS_THREADS / L) + threadIdx.x / L;
+  const int t0 = blockIdx.x * tokens, n = min(tokens, p.n_tokens - t0);
+  if (threadIdx.x < n) {
+    facts[threadIdx.x] = heads_token(p, t0 + threadIdx.x);
+    temp[threadIdx.x] = heads_temperature(p, facts[threadIdx.x].pos);
+  }
+  __syncthreads();
+  constexpr int GROUPS = HS_THREADS / L;
   const int c = threadIdx.x & (L - 1);                      // this lane's chunk of eight
-  const bool live = item < (long)p.n_tokens * p.units;      // a warp's lanes stay together for the exchanges below
-  const HeadsUnit<T> u = heads_unit(p, live ? item : 0);
   const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-  const T* src = p.qkv + (size_t)u.t * p.qkv_stride + u.col;
-  const int CH = p.dk / 8;
-  const bool mine = live && u.kind != 2 && c < CH;
-  if (live && u.kind == 2 && u.dst) {
-    for (int x = c; x < p.row / 8; x += L) {
-      float v[8];
-      if (x < p.dv / 8) {
-        nhv_load8(v, src + x * 8);
-        nhv_store8(u.dst + x * 8, v);
-      } else {
-        nhv_store8(u.dst + x * 8, zero);
-      }
-    }
-  }
-  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-  if (mine) {
-    if (p.taps) {
-      const HeadsPast past = heads_past(p, u.t);
-      const int C = (p.nq + p.nkv) * p.maps * p.dk, at = u.col + c * 8;
-      for (int j = 0; j < p.K; ++j) {
-        const int back = p.K - 1 - j;
-        float x[8], w[8];
-        if (past.before >= back) nhv_load8(x, src - (size_t)back * p.qkv_stride + c * 8);
-        else if (past.has_past) nhv_load8(x, past.state + (size_t)(p.K - 1 + past.before - back) * C + at);
-        else continue;
-        nhv_load8(w, p.taps + (size_t)j * C + at);
+  const int CH = p.dk / 8, C = (p.nq + p.nkv) * p.maps * p.dk;
+  const int half = p.rotary_dim >> 1, hc = half / 8;
+  const bool first = c < hc, turns = c < 2 * hc;
+  const int partner = turns ? (first ? c + hc : c - hc) : c, i0 = (first ? c : c - hc) * 8;
+  for (int base = blockIdx.y * GROUPS; base < p.units; base += gridDim.y * GROUPS) {
+    const int x = base + threadIdx.x / L;
+    const bool live = x < p.units;                          // a warp's lanes stay together for the exchanges below
+    const int kind = x < p.nq * p.maps ? 0 : x < (p.nq + p.nkv) * p.maps ? 1 : 2;
+    const bool mine = live && kind != 2 && c < CH;
+    const int at = x * p.dk + c * 8;                        // the first of this lane's channels (queries and keys)
+    float tap[TAPS > 0 ? TAPS : 1][8];
+    if constexpr (TAPS > 0) {
+      if (mine)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = fmaf(w[e], x[e], v[e]);
-      }
-      if (past.single && past.state && p.K > 1) {           // the only reader of these channels of this state
-        float x[8];
-        for (int j = 0; j + 2 < p.K; ++j) {
-          if (past.has_past) {
-            nhv_load8(x, past.state + (size_t)(j + 1) * C + at);
-            nhv_store8(past.state + (size_t)j * C + at, x);
-          } else {
-            nhv_store8(past.state + (size_t)j * C + at, zero);
+        for (int j = 0; j < TAPS; ++j)                      // the filter right-aligned: the newest token's tap is the last
+          if (j >= TAPS - p.K) nhv_load8(tap[j], p.taps + (size_t)(j - (TAPS - p.K)) * C + at);
+    }
+    float hw[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+    {
+      const T* w = kind == 0 ? p.q_weight : p.k_weight;
+      if (mine && w) nhv_load8(hw, w + c * 8);
+    }
+    for (int i = 0; i < n; ++i) {
+      const int t = t0 + i;
+      const HeadsToken& k = facts[i];
+      const HeadsUnit<T> u = heads_unit(p, t, k, live ? x : 0);
+      const T* src = p.qkv + (size_t)t * p.qkv_stride + u.col;
+      if (kind == 2) {                                      // a value head as it is, the rest of its row cleared
+        if (live && u.dst)
+          for (int y = c; y < p.row / 8; y += L) {
+            float v[8];
+            if (y < p.dv / 8) {
+              nhv_load8(v, src + y * 8);
+              nhv_store8(u.dst + y * 8, v);
+            } else {
+              nhv_store8(u.dst + y * 8, zero);
+            }
           }
-        }
-        nhv_load8(x, src + c * 8);
-        nhv_store8(past.state + (size_t)(p.K - 2) * C + at, x);
       }
-    } else {
-      nhv_load8(v, src + c * 8);
-    }
-    if (u.dst_v) nhv_store8(u.dst_v + c * 8, v);
-  }
-  if (live && u.kind == 1 && u.dst_v)
-    for (int x = CH + c; x < p.row / 8; x += L) nhv_store8(u.dst_v + x * 8, zero);
-  if (p.eps >= 0.f) {
-    float ss = 0.f;
+      float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (mine) {
+        if constexpr (TAPS != 0) {
+          auto past = [&](float (&o)[8], int back) {        // the input `back` tokens before t; false: before the request
+            if (k.before >= back) nhv_load8(o, src - (size_t)back * p.qkv_stride + c * 8);
+            else if (k.has_past) nhv_load8(o, k.state + (size_t)(p.K - 1 + k.before - back) * C + at);
+            else return false;
+            return true;
+          };
+          if constexpr (TAPS > 0) {
+            float in[TAPS][8];
+            bool there[TAPS];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+            for (int j = 0; j < TAPS; ++j) there[j] = j >= TAPS - p.K && past(in[j], TAPS - 1 - j);
 #pragma unroll
-    for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float r = 1.0f / sqrtf(ss / (float)p.dk + p.eps);
-    const T* hw = u.kind == 0 ? p.q_weight : p.k_weight;
-    if (mine) {
-      float w[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
-      if (hw) nhv_load8(w, hw + c * 8);
+            for (int j = 0; j < TAPS; ++j)
+              if (there[j])
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[e] = v[e] * r * w[e];
-    }
-  }
-  const float* cs = heads_angles(p, u.pos);
-  if (cs) {
-    const int half = p.rotary_dim >> 1, hc = half / 8;
-    const bool first = c < hc, turns = c < 2 * hc;
-    const int partner = turns ? (first ? c + hc : c - hc) : c;
-    float co[8], si[8];
-    const int i0 = (first ? c : c - hc) * 8;
-    if (mine && turns) {
-      nhv_load8(co, cs + i0);
-      nhv_load8(si, cs + half + i0);
-    }
+                for (int e = 0; e < 8; ++e) v[e] = fmaf(tap[j][e], in[j][e], v[e]);
+          } else {
+            for (int j = 0; j < p.K; ++j) {
+              float in[8], w[8];
+              if (!past(in, p.K - 1 - j)) continue;
+              nhv_load8(w, p.taps + (size_t)j * C + at);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      const float other = __shfl_sync(0xffffffffu, v[e], partner, L);
-      if (mine && turns) v[e] = first ? v[e] * co[e] - other * si[e] : v[e] * co[e] + other * si[e];
-    }
-  }
-  if (!live || u.kind == 2 || !u.dst) return;
-  const int from = u.map * CH;
-  if (mine) {
-    if (u.kind == 0 && p.temp_every > 0) {
-      const float f = heads_temperature(p, u.pos);
+              for (int e = 0; e < 8; ++e) v[e] = fmaf(w[e], in[e], v[e]);
+            }
+          }
+          if (k.single && k.state && p.K > 1) {             // the only reader of these channels of this state
+            float in[8];
+            for (int j = 0; j + 2 < p.K; ++j) {
+              if (k.has_past) {
+                nhv_load8(in, k.state + (size_t)(j + 1) * C + at);
+                nhv_store8(k.state + (size_t)j * C + at, in);
+              } else {
+                nhv_store8(k.state + (size_t)j * C + at, zero);
+              }
+            }
+            nhv_load8(in, src + c * 8);
+            nhv_store8(k.state + (size_t)(p.K - 2) * C + at, in);
+          }
+        } else {
+          nhv_load8(v, src + c * 8);
+        }
+        if (u.dst_v) nhv_store8(u.dst_v + c * 8, v);
+      }
+      if (live && kind == 1 && u.dst_v)
+        for (int y = CH + c; y < p.row / 8; y += L) nhv_store8(u.dst_v + y * 8, zero);
+      if (p.eps >= 0.f) {
+        float ss = 0.f;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[e] *= f;
+        for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+#pragma unroll
+        for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float r = 1.0f / sqrtf(ss / (float)p.dk + p.eps);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * r * hw[e];
+      }
+      const float* cs = heads_angles(p, k.pos);
+      if (cs) {
+        float co[8], si[8];
+        if (mine && turns) {
+          nhv_load8(co, cs + i0);
+          nhv_load8(si, cs + half + i0);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float other = __shfl_sync(0xffffffffu, v[e], partner, L);
+          if (mine && turns) v[e] = first ? v[e] * co[e] - other * si[e] : v[e] * co[e] + other * si[e];
+        }
+      }
+      if (!live || kind == 2 || !u.dst) continue;           // no exchange from here on
+      const int from = u.map * CH;
+      if (mine) {
+        if (kind == 0) {
+          const float f = temp[i];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[e] *= f;
+        }
+        nhv_store8(u.dst + (from + c) * 8, v);
+      }
+      if (kind == 0) {
+        for (int y = c; y < p.q_head / 8; y += L)
+          if (y < from || y >= from + CH) nhv_store8(u.dst + y * 8, zero);
+      } else if (u.map == p.maps - 1) {
+        for (int y = p.maps * CH + c; y < p.row / 8; y += L) nhv_store8(u.dst + y * 8, zero);
+      }
     }
-    nhv_store8(u.dst + (from + c) * 8, v);
-  }
-  if (u.kind == 0) {
-    for (int x = c; x < p.q_head / 8; x += L)
-      if (x < from || x >= from + CH) nhv_store8(u.dst + x * 8, zero);
-  } else if (u.map == p.maps - 1) {
-    for (int x = p.maps * CH + c; x < p.row / 8; x += L) nhv_store8(u.dst + x * 8, zero);
   }
 }
 
@@ -237,8 +295,10 @@ __global__ void __launch_bounds__(HS_WARPS * 32) heads_store_kernel(const HeadsS
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long item = (long)blockIdx.x * HS_WARPS + warp;
   if (item >= (long)p.n_tokens * p.units) return;
-  const HeadsUnit<T> u = heads_unit(p, item);
-  const T* src = p.qkv + (size_t)u.t * p.qkv_stride + u.col;
+  const int t = (int)(item / p.units);
+  const HeadsToken k = heads_token(p, t);
+  const HeadsUnit<T> u = heads_unit(p, t, k, (int)(item - (long)t * p.units));
+  const T* src = p.qkv + (size_t)t * p.qkv_stride + u.col;
   if (u.kind == 2) {
     if (u.dst)
       for (int c = lane; c < p.row; c += 32) u.dst[c] = c < p.dv ? src[c] : from_f32<T>(0.f);
@@ -247,7 +307,6 @@ __global__ void __launch_bounds__(HS_WARPS * 32) heads_store_kernel(const HeadsS
   float* v = smem + (size_t)warp * p.dk;
   const int d = p.dk;
   if (p.taps) {
-    const HeadsPast past = heads_past(p, u.t);
     const int C = (p.nq + p.nkv) * p.maps * d;
     for (int c = lane; c < d; c += 32) {
       const int at = u.col + c;
@@ -255,16 +314,16 @@ __global__ void __launch_bounds__(HS_WARPS * 32) heads_store_kernel(const HeadsS
       for (int j = 0; j < p.K; ++j) {
         const int back = p.K - 1 - j;
         float x;
-        if (past.before >= back) x = to_f32<T>(*(src + c - (size_t)back * p.qkv_stride));
-        else if (past.has_past) x = past.state[(size_t)(p.K - 1 + past.before - back) * C + at];
+        if (k.before >= back) x = to_f32<T>(*(src + c - (size_t)back * p.qkv_stride));
+        else if (k.has_past) x = k.state[(size_t)(p.K - 1 + k.before - back) * C + at];
         else continue;
         acc = fmaf(to_f32<T>(p.taps[(size_t)j * C + at]), x, acc);
       }
       v[c] = acc;
-      if (past.single && past.state && p.K > 1) {
+      if (k.single && k.state && p.K > 1) {
         for (int j = 0; j + 2 < p.K; ++j)
-          past.state[(size_t)j * C + at] = past.has_past ? past.state[(size_t)(j + 1) * C + at] : 0.f;
-        past.state[(size_t)(p.K - 2) * C + at] = to_f32<T>(src[c]);
+          k.state[(size_t)j * C + at] = k.has_past ? k.state[(size_t)(j + 1) * C + at] : 0.f;
+        k.state[(size_t)(p.K - 2) * C + at] = to_f32<T>(src[c]);
       }
     }
   } else {
@@ -281,9 +340,9 @@ __global__ void __launch_bounds__(HS_WARPS * 32) heads_store_kernel(const HeadsS
   }
   __syncwarp();
   if (!u.dst) return;
-  const float* cs = heads_angles(p, u.pos);
+  const float* cs = heads_angles(p, k.pos);
   const int half = p.rotary_dim >> 1, from = u.map * d;
-  const float f = u.kind == 0 ? heads_temperature(p, u.pos) : 1.0f;
+  const float f = u.kind == 0 ? heads_temperature(p, k.pos) : 1.0f;
   for (int c = lane; c < d; c += 32) {
     float y = v[c];
     if (cs && c < half) y = v[c] * cs[c] - v[c + half] * cs[half + c];
@@ -328,13 +387,24 @@ static int heads_store_launch(HeadsStore<T> p, bool portions, cudaStream_t strea
                    (!p.taps || p.K < 2 || p.state_stride % 4 == 0) && ok16(p.qkv) && ok16(p.q_out) && ok16(p.kv_pages) &&
                    ok16(p.q_weight) && ok16(p.k_weight) && ok16(p.taps) && ok16(p.state);
   if (vec) {
-    const int ch = p.dk / 8;
-#define GO(L)                                                                                               \
-  nhv_launch(heads_store_vec_kernel<T, L>, (unsigned)((items + HS_THREADS / L - 1) / (HS_THREADS / L)), HS_THREADS, 0, stream, p)
-    if (ch <= 4) GO(4);
-    else if (ch <= 8) GO(8);
-    else if (ch <= 16) GO(16);
-    else GO(32);
+    const int ch = p.dk / 8, L = ch <= 4 ? 4 : ch <= 8 ? 8 : ch <= 16 ? 16 : 32;
+    // long steps: several tokens a block, so that a unit's taps and weights are read once for them; short steps: a block
+    // per share of a token's units
+    const int tokens = p.n_tokens >= 2048 ? HS_TOKENS : 1;
+    const int blocks = (p.n_tokens + tokens - 1) / tokens, passes = (p.units + HS_THREADS / L - 1) / (HS_THREADS / L);
+    const dim3 grid(blocks, blocks >= 592 ? 1 : passes);
+#define GO(L, TAPS) nhv_launch(heads_store_vec_kernel<T, L, TAPS>, grid, HS_THREADS, 0, stream, p, tokens)
+#define PICK(L)                                  \
+  do {                                           \
+    if (!p.taps) GO(L, 0);                       \
+    else if (p.K <= HS_TAPS) GO(L, HS_TAPS);     \
+    else GO(L, -1);                              \
+  } while (0)
+    if (L == 4) PICK(4);
+    else if (L == 8) PICK(8);
+    else if (L == 16) PICK(16);
+    else PICK(32);
+#undef PICK
 #undef GO
   } else {
     const size_t smem = (size_t)HS_WARPS * p.dk * sizeof(float);
@@ -350,14 +420,15 @@ static int heads_store_launch(HeadsStore<T> p, bool portions, cudaStream_t strea
   return 0;
 }
 
-// portions != 0: some request of the step brings more than one token.
+// portions != 0: some request of the step brings more than one token; one_each != 0: every request brings exactly one (so
+// that token t is request t's).
 NHV_API int nhv_heads_store(int dtype, const void* qkv, int qkv_stride, void* q_out, int q_out_stride, int q_head,
                             void* kv_pages, const int* slot_mapping, const int* positions, const float* cos_sin,
                             int rotary_dim, int max_position, int n_tokens, int nq, int nkv, int maps, int dk, int dv,
                             int row, int page_size, int n_pages, float eps, const void* q_weight, const void* k_weight,
                             int v_from_k, float temp_coef, int temp_every, const void* taps, int K, float* state,
                             long state_stride, const int* cu_q, const int* q_start, const int* slots, int n_seqs,
-                            int portions, cudaStream_t stream) {
+                            int portions, int one_each, cudaStream_t stream) {
   if (n_tokens == 0 || n_seqs == 0) return 0;
   NHV_REQUIRE(n_tokens > 0 && nq > 0 && nkv >= 0 && maps > 0 && dk > 0 && dv > 0, "heads_store: bad sizes");
   NHV_REQUIRE(dk <= 2048, "heads_store: a head of %d elements is beyond the supported 2048", dk);
@@ -377,7 +448,7 @@ NHV_API int nhv_heads_store(int dtype, const void* qkv, int qkv_stride, void* q_
       HeadsStore<T>{(const T*)qkv, (T*)q_out, (T*)kv_pages, (const T*)q_weight, (const T*)k_weight, (const T*)taps,  \
                     state, slot_mapping, positions, cu_q, q_start, slots, cos_sin, state_stride, qkv_stride,         \
                     q_out_stride, q_head, cos_sin ? rotary_dim : 0, max_position, n_tokens, n_seqs, nq, nkv, maps,   \
-                    dk, dv, row, page_size, n_pages, K, v_from_k, units, temp_every, eps, temp_coef},                \
+                    dk, dv, row, page_size, n_pages, K, v_from_k, units, temp_every, one_each, eps, temp_coef},      \
       portions != 0, stream)
   if (dtype == NHV_F32) GO(float);
   if (dtype == NHV_BF16) GO(__nv_bfloat16);

@@ -139,21 +139,34 @@ __host__ __device__ __forceinline__ int nhv_first_key(int pos, int window, int c
   return lo;
 }
 
-// Scores capped smoothly, cap * tanh(raw * scale / cap), in log2 units: cap * log2(e) * (1 - 2 / (1 + e^(2 z))) with
-// z = raw * scale / cap, so that exp2 of it is the exponential of the capped score.  `in` = 2 log2(e) scale / cap turns a
-// raw score into the exponent of 2, `out` = cap log2(e).  Two scores share one reciprocal (of the product of both
-// denominators, whose exponents are kept below 2^60 so that it cannot overflow: tanh is 1 to the last bit long before).
-// The error is a few units of 2^-24 of the cap.
+// Scores capped smoothly, cap * tanh(z) with z = raw * scale / cap, in log2 units, so that exp2 of it is the exponential of
+// the capped score.  Two forms, chosen by a warp for a whole tile of scores:
+//   small scores (|z| <= 1/2 throughout): z times a polynomial in z^2, the least worst error over that range (3e-9; fitted
+//     to tanh(z) / z by least squares on Chebyshev points, reweighted by the error), multiply-adds only;
+//   else cap log2(e) (1 - 2 / (1 + e^(2 z))): `in` = 2 log2(e) scale / cap turns a raw score into the exponent of 2.  Two
+//     scores share one reciprocal (of the product of both denominators, whose exponents are kept below 2^60 so that it
+//     cannot overflow: tanh is 1 to the last bit long before).
+// The error is a few units of 2^-24 of the cap in both.
 struct NhvScoreCap {
-  float in, out;      // in == 0: scores are not capped
+  float in, out;        // in == 0: scores are not capped; out = cap log2(e)
+  float z, small;       // scale / cap; the raw score at |z| = 1/2
+  float c[5];           // the polynomial's coefficients times out
 };
 inline NhvScoreCap nhv_score_cap(float scale, float cap) {
-  NhvScoreCap c = {0.f, 0.f};
+  NhvScoreCap c = {};
   if (cap > 0.f) {
+    const float tanh_over_z[5] = {0.9999999312f, -0.3333277586f, 0.1332057123f, -0.05276213199f, 0.01673756908f};
     c.in = 2.0f * 1.4426950408889634f * scale / cap;
     c.out = cap * 1.4426950408889634f;
+    c.z = scale / cap;
+    c.small = 0.5f * cap / (scale < 0.f ? -scale : scale);
+    for (int i = 0; i < 5; ++i) c.c[i] = tanh_over_z[i] * c.out;
   }
   return c;
+}
+__device__ __forceinline__ float nhv_cap_small(float raw, const NhvScoreCap& c) {
+  const float z = raw * c.z, t = z * z;
+  return z * fmaf(fmaf(fmaf(fmaf(c.c[4], t, c.c[3]), t, c.c[2]), t, c.c[1]), t, c.c[0]);
 }
 __device__ __forceinline__ void nhv_cap_scores(float& a, float& b, const NhvScoreCap& c) {
   float ea, eb, r;
@@ -165,6 +178,26 @@ __device__ __forceinline__ void nhv_cap_scores(float& a, float& b, const NhvScor
   r *= -2.0f * c.out;
   a = fmaf(r, eb, c.out);
   b = fmaf(r, ea, c.out);
+}
+// The scores of a warp's tile, N groups of four a thread (scores that a mask replaces later may be anything).
+template <int N>
+__device__ __forceinline__ void nhv_cap_tile(float (&s)[N][4], const NhvScoreCap& c) {
+  float m = 0.f;
+#pragma unroll
+  for (int j = 0; j < N; ++j)
+    m = fmaxf(fmaxf(m, fmaxf(fabsf(s[j][0]), fabsf(s[j][1]))), fmaxf(fabsf(s[j][2]), fabsf(s[j][3])));
+  if (__all_sync(0xffffffffu, m <= c.small)) {
+#pragma unroll
+    for (int j = 0; j < N; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[j][e] = nhv_cap_small(s[j][e], c);
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      nhv_cap_scores(s[j][0], s[j][1], c);
+      nhv_cap_scores(s[j][2], s[j][3], c);
+    }
+  }
 }
 
 template <typename T> __device__ __forceinline__ float to_f32(T v);

@@ -149,8 +149,8 @@ NHV_API int nhv_sandwich_stream(int dtype, void* out, float* stream_rows, const 
   return 0;
 }
 
-template <typename T>
-__global__ void embed_rmsnorm_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(512) embed_rmsnorm_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
                                      const T* __restrict__ w, int width, int vocab, float eps, float offset) {
   __shared__ float red[33];
   pdl_prologue();
@@ -158,11 +158,31 @@ __global__ void embed_rmsnorm_kernel(float* __restrict__ out, const T* __restric
   const bool ok = id >= 0 && id < vocab;
   const T* src = table + (size_t)(ok ? id : 0) * width;
   float ss = 0.f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = to_f32<T>(src[c]);
-    ss = fmaf(v, v, ss);
+  if constexpr (VEC) {
+    for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+      float v[8];
+      nhv_load8(v, src + c);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float v = to_f32<T>(src[c]);
+      ss = fmaf(v, v, ss);
+    }
   }
   const float r = ok ? 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps) : 0.f;      // an id outside the table: zeros
+  if constexpr (VEC) {
+    for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+      float v[8], wv[8];
+      nhv_load8(v, src + c);                                  // from the cache: the row was just read
+      nhv_load8(wv, w + c);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = v[e] * r * (wv[e] + offset);
+      nhv_store8(out + (size_t)t * width + c, v);
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < width; c += blockDim.x)
     out[(size_t)t * width + c] = to_f32<T>(src[c]) * r * (to_f32<T>(w[c]) + offset);
 }
@@ -171,12 +191,13 @@ NHV_API int nhv_embed_rmsnorm(int dtype, float* out, const void* table, const in
                               int vocab, float eps, float offset, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   NHV_REQUIRE(n_tokens > 0 && width > 0 && vocab > 0, "embed_rmsnorm: bad sizes");
+  const bool vec = width % 8 == 0 && sw_aligned(out) && sw_aligned(table) && sw_aligned(w);
   int threads = 32;
-  while (threads < 512 && threads * 4 < width) threads <<= 1;
-#define GO(T)                                                                                                        \
-  nhv_launch(embed_rmsnorm_kernel<T>, n_tokens, threads, 0, stream, out, (const T*)table, ids, (const T*)w, width, vocab, eps, offset)
-  if (dtype == NHV_F32) GO(float);
-  else if (dtype == NHV_BF16) GO(__nv_bfloat16);
+  while (threads < 512 && threads * (vec ? 8 : 4) < width) threads <<= 1;
+#define GO(T, V)                                                                                                     \
+  nhv_launch(embed_rmsnorm_kernel<T, V>, n_tokens, threads, 0, stream, out, (const T*)table, ids, (const T*)w, width, vocab, eps, offset)
+  if (dtype == NHV_F32) { if (vec) GO(float, true); else GO(float, false); }
+  else if (dtype == NHV_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
   else NHV_REQUIRE(false, "embed_rmsnorm: unknown dtype %d", dtype);
 #undef GO
   NHV_CHECK_LAUNCH("embed_rmsnorm");

@@ -228,13 +228,7 @@ __device__ __forceinline__ void warp_half_tile(RowState& st, const uint32_t (&qf
       mma_bf16(s[j + 1], qf[k], b[2], b[3]);
     }
   }
-  if (cap.in != 0.f) {                                         // capped scores are in log2 units: scale_log2 is 1 then
-#pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      nhv_cap_scores(s[j][0], s[j][1], cap);
-      nhv_cap_scores(s[j][2], s[j][3], cap);
-    }
-  }
+  if (cap.in != 0.f) nhv_cap_tile<NT>(s, cap);                 // capped scores are in log2 units: scale_log2 is 1 then
   float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
   for (int j = 0; j < NT; ++j) {

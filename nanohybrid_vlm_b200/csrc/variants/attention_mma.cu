@@ -157,13 +157,7 @@ __device__ __forceinline__ void warp_tile(RowState& st, const uint32_t (&qf)[KS]
       mma_bf16(s[j + 1], qf[k], b[2], b[3]);
     }
   }
-  if (cap.in != 0.f) {                                         // capped scores are in log2 units: scale_log2 is 1 then
-#pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      nhv_cap_scores(s[j][0], s[j][1], cap);
-      nhv_cap_scores(s[j][2], s[j][3], cap);
-    }
-  }
+  if (cap.in != 0.f) nhv_cap_tile<NT>(s, cap);                 // capped scores are in log2 units: scale_log2 is 1 then
   // mask and the tile's row maxima
   float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -285,12 +279,7 @@ __device__ __forceinline__ void warp_tile_prefill(PrefillState<MTW>& st, const b
     }
     if (cap.in != 0.f) {
 #pragma unroll
-      for (int mt = 0; mt < MTW; ++mt)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          nhv_cap_scores(s[mt][j][0], s[mt][j][1], cap);
-          nhv_cap_scores(s[mt][j][2], s[mt][j][3], cap);
-        }
+      for (int mt = 0; mt < MTW; ++mt) nhv_cap_tile<4>(s[mt], cap);
     }
     uint32_t pf[MTW][2][4];
 #pragma unroll

@@ -183,6 +183,37 @@ struct alignas(64) Params {
   NhvScoreCap cap;        // in == 0: none
 };
 
+// A row's scores capped (see nhv_cap_tile), two at a time in packed arithmetic where they are small.
+__device__ __forceinline__ void cap_row(uint32_t (&sr)[2][32], const NhvScoreCap& c) {
+  float m0 = 0.f, m1 = 0.f;
+#pragma unroll
+  for (int i = 0; i < BN; i += 4) {
+    m0 = max3(m0, fabsf(__uint_as_float(sr[i >> 5][i & 31])), fabsf(__uint_as_float(sr[i >> 5][(i & 31) + 1])));
+    m1 = max3(m1, fabsf(__uint_as_float(sr[i >> 5][(i & 31) + 2])), fabsf(__uint_as_float(sr[i >> 5][(i & 31) + 3])));
+  }
+  if (__all_sync(0xffffffffu, fmaxf(m0, m1) <= c.small)) {
+    const f32x2 z2 = f2_pack(c.z, c.z), k0 = f2_pack(c.c[0], c.c[0]), k1 = f2_pack(c.c[1], c.c[1]), k2 = f2_pack(c.c[2], c.c[2]),
+                k3 = f2_pack(c.c[3], c.c[3]), k4 = f2_pack(c.c[4], c.c[4]);
+#pragma unroll
+    for (int i = 0; i < BN; i += 2) {
+      const f32x2 z = f2_mul(f2_pack(__uint_as_float(sr[i >> 5][i & 31]), __uint_as_float(sr[i >> 5][(i & 31) + 1])), z2);
+      const f32x2 t = f2_mul(z, z);
+      float a, b;
+      f2_unpack(f2_mul(z, f2_fma(f2_fma(f2_fma(f2_fma(k4, t, k3), t, k2), t, k1), t, k0)), a, b);
+      sr[i >> 5][i & 31] = __float_as_uint(a);
+      sr[i >> 5][(i & 31) + 1] = __float_as_uint(b);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < BN; i += 2) {
+      float a = __uint_as_float(sr[i >> 5][i & 31]), b = __uint_as_float(sr[i >> 5][(i & 31) + 1]);
+      nhv_cap_scores(a, b, c);
+      sr[i >> 5][i & 31] = __float_as_uint(a);
+      sr[i >> 5][(i & 31) + 1] = __float_as_uint(b);
+    }
+  }
+}
+
 __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tcgen05_kernel(const __grid_constant__ Params p) {
   extern __shared__ __align__(128) unsigned char smem_raw[];
   // barriers in the first 128 bytes, the tiles from the next 1024-byte boundary on
@@ -388,15 +419,7 @@ __global__ void __launch_bounds__(THREADS, (2 * BN + DV) <= 256 ? 2 : 1) attn_tc
       // and the scaling folded into the exponent's multiply-add.  A tile that some row of the block sees only
       // in part takes the masked path.
       const bool masked = !(key_base >= all_lo && key_base + BN - 1 <= all_hi);
-      if (p.cap.in != 0.f) {
-#pragma unroll
-        for (int i = 0; i < BN; i += 2) {
-          float a = __uint_as_float(sr[i >> 5][i & 31]), b = __uint_as_float(sr[i >> 5][(i & 31) + 1]);
-          nhv_cap_scores(a, b, p.cap);
-          sr[i >> 5][i & 31] = __float_as_uint(a);
-          sr[i >> 5][(i & 31) + 1] = __float_as_uint(b);
-        }
-      }
+      if (p.cap.in != 0.f) cap_row(sr, p.cap);
       if (p.slopes) {                                           // score - slope * (row - key), before maximum and mask
         const float at0 = slope * (float)(key_base - row_hi);
 #pragma unroll

@@ -78,7 +78,7 @@ _SIGNATURES = {
     "nhv_streams_rmsnorm": [I, P, P, P, I, P, P, P, P, P, P, I, I, I, F, P],
     "nhv_row_norm_store": [I, P, I, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P, I, P, P],
     "nhv_heads_store": [I, P, I, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P, I, F, I, P, I, P, ctypes.c_long,
-                        P, P, P, I, I, P],
+                        P, P, P, I, I, I, P],
     "nhv_map_difference": [I, P, I, P, I, P, F, F, I, I, I, P],
     "nhv_sandwich_stream": [I, P, P, P, P, P, P, I, I, F, F, F, F, I, P],
     "nhv_embed_rmsnorm": [I, P, P, P, P, I, I, I, F, F, P],

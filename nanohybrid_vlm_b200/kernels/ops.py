@@ -937,7 +937,8 @@ def heads_store(qkv, q_out, q_head: int, kv_pages, slot_mapping, batch, cos_sin,
          0 if cos_sin is None else cos_sin.shape[0], T, nq, nkv, int(maps), dk, dv, row, page_size, n_pages,
          -1.0 if eps is None else float(eps), _ptr(q_weight), _ptr(k_weight), int(bool(values_from_keys)), float(coef),
          int(every), _ptr(taps), K, _ptr(state) if K > 1 else None, state.stride(0) if K > 1 else 0, batch.cu_q.data_ptr(),
-         batch.q_start.data_ptr(), batch.state_slots.data_ptr(), batch.n_seqs, int(batch.n_prefill_seqs > 0), stream_ptr())
+         batch.q_start.data_ptr(), batch.state_slots.data_ptr(), batch.n_seqs, int(batch.n_prefill_seqs > 0),
+         int(batch.n_prefill_seqs == 0 and T == batch.n_seqs), stream_ptr())
 
 
 def map_difference(out, a, share, factor: float, eps: float, heads: int, dv: int) -> None:
