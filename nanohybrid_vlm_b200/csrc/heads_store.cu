@@ -26,9 +26,13 @@
 #include "nhv_common.cuh"
 #include "nhv_vec8.cuh"
 
-constexpr int HS_THREADS = 256;
-constexpr int HS_TOKENS = 4;             // the most tokens of a block
-constexpr int HS_TAPS = 4;               // filters of up to so many taps keep theirs in registers
+// Measured on B200 (4,096 tokens, 64 maps of 64 over 8 KV heads): what counts is how many warps an SM holds; more units or
+// tokens per thread cost registers and lose (blocks of 256 with 3 units a thread: 94 us, these: 61 us).
+constexpr int HS_THREADS = 128;
+constexpr int HS_BLOCKS = 6;             // on an SM at least
+constexpr int HS_BATCH = 2;              // units whose elements a thread asks for at once (no filter)
+constexpr int HS_TOKENS = 2;             // tokens of a block in long steps (filters)
+constexpr int HS_TAPS = 4;               // filters of up to so many taps run eight elements a lane
 constexpr int HS_WARPS = 4;              // of the general kernel
 
 template <typename T>
@@ -140,149 +144,226 @@ __device__ __forceinline__ const float* heads_angles(const HeadsStore<T>& p, int
   return p.cos_sin + (size_t)pos * p.rotary_dim;
 }
 
-// L lanes per unit, eight consecutive elements a lane: sizes in steps of 8, halves of the rotation too.  A block takes
-// `tokens` neighbouring tokens (gridDim.x) and all their units, or a share of them (gridDim.y); a unit's filter taps are read
-// once for its tokens.  TAPS: taps held in registers (0: no filter; filters of more taps read theirs per token, TAPS -1).
-template <typename T, int L, int TAPS>
-__global__ void __launch_bounds__(HS_THREADS) heads_store_vec_kernel(const HeadsStore<T> p, int tokens) {
-  __shared__ HeadsToken facts[HS_TOKENS];
-  __shared__ float temp[HS_TOKENS];
+// Eight elements as they lie in memory (so that many can be on their way in few registers), and as floats.
+template <typename T>
+struct Raw8 { uint4 w[sizeof(T) / 2]; };
+template <typename T>
+__device__ __forceinline__ void raw_load(Raw8<T>& r, const T* src) {
+#pragma unroll
+  for (int i = 0; i < (int)(sizeof(T) / 2); ++i) r.w[i] = reinterpret_cast<const uint4*>(src)[i];
+}
+template <typename T>
+__device__ __forceinline__ void raw_get(float (&v)[8], const Raw8<T>& r) { nhv_load8(v, reinterpret_cast<const T*>(r.w)); }
+
+// Norm, rotation, temperature and the store of one unit's chunk of eight; all lanes of a warp come here together.
+// mine: this lane holds elements of a query or key; co / si: its cosines and sines (turns: its elements rotate).
+struct HeadsLane {
+  int c, partner, i0;
+  bool first, turns;
+};
+template <typename T, int L>
+__device__ __forceinline__ void heads_finish(const HeadsStore<T>& p, float (&v)[8], const HeadsUnit<T>& u, bool live, bool mine,
+                                             const HeadsLane& lane, const float (&hw)[8], bool rotate, const float (&co)[8],
+                                             const float (&si)[8], float temp) {
+  const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  const int CH = p.dk / 8, c = lane.c;
+  if (p.eps >= 0.f) {
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float r = 1.0f / sqrtf(ss / (float)p.dk + p.eps);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = v[e] * r * hw[e];
+  }
+  if (rotate) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float other = __shfl_sync(0xffffffffu, v[e], lane.partner, L);
+      if (mine && lane.turns) v[e] = lane.first ? v[e] * co[e] - other * si[e] : v[e] * co[e] + other * si[e];
+    }
+  }
+  if (!live || u.kind == 2 || !u.dst) return;
+  const int from = u.map * CH;
+  if (mine) {
+    if (u.kind == 0) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= temp;
+    }
+    nhv_store8(u.dst + (from + c) * 8, v);
+  }
+  if (u.kind == 0) {
+    for (int y = c; y < p.q_head / 8; y += L)
+      if (y < from || y >= from + CH) nhv_store8(u.dst + y * 8, zero);
+  } else if (u.map == p.maps - 1) {
+    for (int y = p.maps * CH + c; y < p.row / 8; y += L) nhv_store8(u.dst + y * 8, zero);
+  }
+}
+
+template <typename T, int L>
+__device__ __forceinline__ HeadsLane heads_lane(const HeadsStore<T>& p) {
+  HeadsLane l;
+  l.c = threadIdx.x & (L - 1);
+  const int hc = (p.rotary_dim >> 1) / 8;
+  l.first = l.c < hc;
+  l.turns = l.c < 2 * hc;
+  l.partner = l.turns ? (l.first ? l.c + hc : l.c - hc) : l.c;
+  l.i0 = (l.first ? l.c : l.c - hc) * 8;
+  return l;
+}
+
+// L lanes per unit, eight consecutive elements a lane: sizes in steps of 8, halves of the rotation too.
+
+// Without a filter: a block per token (gridDim.x) and its units, or a share of them (gridDim.y); HS_BATCH of a thread's units
+// are read before the first is worked on, its angles once for all of them.
+template <typename T, int L>
+__global__ void __launch_bounds__(HS_THREADS, HS_BLOCKS) heads_store_vec_kernel(const HeadsStore<T> p) {
   pdl_prologue();
-  const int t0 = blockIdx.x * tokens, n = min(tokens, p.n_tokens - t0);
+  constexpr int GROUPS = HS_THREADS / L;
+  const int t = blockIdx.x;
+  const HeadsToken k = heads_token(p, t);
+  const float temp = heads_temperature(p, k.pos);
+  const HeadsLane lane = heads_lane<T, L>(p);
+  const int c = lane.c, CH = p.dk / 8, step = gridDim.y * GROUPS;
+  const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  const T* row = p.qkv + (size_t)t * p.qkv_stride;
+  const float* cs = heads_angles(p, k.pos);
+  float co[8], si[8];
+  if (cs && lane.turns && c < CH) {
+    nhv_load8(co, cs + lane.i0);
+    nhv_load8(si, cs + (p.rotary_dim >> 1) + lane.i0);
+  }
+  for (int base = blockIdx.y * GROUPS; base < p.units; base += HS_BATCH * step) {
+    Raw8<T> raw[HS_BATCH];
+#pragma unroll
+    for (int b = 0; b < HS_BATCH; ++b) {
+      const int x = base + b * step + threadIdx.x / L;
+      if (x < (p.nq + p.nkv) * p.maps && x < p.units && c < CH) raw_load(raw[b], row + (size_t)x * p.dk + c * 8);
+    }
+#pragma unroll
+    for (int b = 0; b < HS_BATCH; ++b) {
+      if (base + b * step >= p.units) break;                // the same for the whole block
+      const int x = base + b * step + threadIdx.x / L;
+      const bool live = x < p.units;
+      const HeadsUnit<T> u = heads_unit(p, t, k, live ? x : 0);
+      const bool mine = live && u.kind != 2 && c < CH;
+      float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      float hw[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+      if (mine) {
+        raw_get(v, raw[b]);
+        const T* w = u.kind == 0 ? p.q_weight : p.k_weight;
+        if (w) nhv_load8(hw, w + c * 8);
+        if (u.dst_v) nhv_store8(u.dst_v + c * 8, v);
+      }
+      if (live && u.kind == 1 && u.dst_v)
+        for (int y = CH + c; y < p.row / 8; y += L) nhv_store8(u.dst_v + y * 8, zero);
+      if (live && u.kind == 2 && u.dst)                     // a value head as it is, the rest of its row cleared
+        for (int y = c; y < p.row / 8; y += L) {
+          float val[8];
+          if (y < p.dv / 8) {
+            nhv_load8(val, row + u.col + y * 8);
+            nhv_store8(u.dst + y * 8, val);
+          } else {
+            nhv_store8(u.dst + y * 8, zero);
+          }
+        }
+      heads_finish<T, L>(p, v, u, live, mine, lane, hw, cs != nullptr, co, si, temp);
+    }
+  }
+}
+
+// With a filter of up to TAPS taps: a block takes NT neighbouring tokens (gridDim.x) and all their units, or a share of them
+// (gridDim.y); a unit's taps are read once for its tokens, and the inputs of all of them (and of the TAPS - 1 tokens before)
+// before the first is worked on.
+template <typename T, int L, int TAPS, int NT>
+__global__ void __launch_bounds__(HS_THREADS, 4) heads_filter_vec_kernel(const HeadsStore<T> p) {
+  __shared__ HeadsToken facts[NT];
+  __shared__ float temps[NT];
+  pdl_prologue();
+  const int t0 = blockIdx.x * NT, n = min(NT, p.n_tokens - t0);
   if (threadIdx.x < n) {
     facts[threadIdx.x] = heads_token(p, t0 + threadIdx.x);
-    temp[threadIdx.x] = heads_temperature(p, facts[threadIdx.x].pos);
+    temps[threadIdx.x] = heads_temperature(p, facts[threadIdx.x].pos);
   }
   __syncthreads();
-  constexpr int GROUPS = HS_THREADS / L;
-  const int c = threadIdx.x & (L - 1);                      // this lane's chunk of eight
+  constexpr int GROUPS = HS_THREADS / L, X = TAPS - 1;
+  const HeadsLane lane = heads_lane<T, L>(p);
+  const int c = lane.c, CH = p.dk / 8, C = (p.nq + p.nkv) * p.maps * p.dk, skip = TAPS - p.K;
   const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-  const int CH = p.dk / 8, C = (p.nq + p.nkv) * p.maps * p.dk;
-  const int half = p.rotary_dim >> 1, hc = half / 8;
-  const bool first = c < hc, turns = c < 2 * hc;
-  const int partner = turns ? (first ? c + hc : c - hc) : c, i0 = (first ? c : c - hc) * 8;
   for (int base = blockIdx.y * GROUPS; base < p.units; base += gridDim.y * GROUPS) {
     const int x = base + threadIdx.x / L;
     const bool live = x < p.units;                          // a warp's lanes stay together for the exchanges below
     const int kind = x < p.nq * p.maps ? 0 : x < (p.nq + p.nkv) * p.maps ? 1 : 2;
     const bool mine = live && kind != 2 && c < CH;
     const int at = x * p.dk + c * 8;                        // the first of this lane's channels (queries and keys)
-    float tap[TAPS > 0 ? TAPS : 1][8];
-    if constexpr (TAPS > 0) {
-      if (mine)
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j)                      // the filter right-aligned: the newest token's tap is the last
-          if (j >= TAPS - p.K) nhv_load8(tap[j], p.taps + (size_t)(j - (TAPS - p.K)) * C + at);
-    }
+    Raw8<T> in[NT + X], tap[TAPS];                          // in[r]: the input of token t0 - X + r; taps right-aligned
     float hw[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
-    {
-      const T* w = kind == 0 ? p.q_weight : p.k_weight;
-      if (mine && w) nhv_load8(hw, w + c * 8);
-    }
-    for (int i = 0; i < n; ++i) {
-      const int t = t0 + i;
-      const HeadsToken& k = facts[i];
-      const HeadsUnit<T> u = heads_unit(p, t, k, live ? x : 0);
-      const T* src = p.qkv + (size_t)t * p.qkv_stride + u.col;
-      if (kind == 2) {                                      // a value head as it is, the rest of its row cleared
-        if (live && u.dst)
-          for (int y = c; y < p.row / 8; y += L) {
-            float v[8];
-            if (y < p.dv / 8) {
-              nhv_load8(v, src + y * 8);
-              nhv_store8(u.dst + y * 8, v);
-            } else {
-              nhv_store8(u.dst + y * 8, zero);
-            }
-          }
+    if (mine) {
+#pragma unroll
+      for (int r = 0; r < NT + X; ++r) {
+        const int t = t0 - X + r;
+        if (r >= skip && t >= 0 && t < t0 + n) raw_load(in[r], p.qkv + (size_t)t * p.qkv_stride + at);
       }
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+        if (j >= skip) raw_load(tap[j], p.taps + (size_t)(j - skip) * C + at);
+      const T* w = kind == 0 ? p.q_weight : p.k_weight;
+      if (w) nhv_load8(hw, w + c * 8);
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      if (i >= n) break;                                    // the same for the whole block
+      const HeadsToken& k = facts[i];
+      const HeadsUnit<T> u = heads_unit(p, t0 + i, k, live ? x : 0);
       float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
       if (mine) {
-        if constexpr (TAPS != 0) {
-          auto past = [&](float (&o)[8], int back) {        // the input `back` tokens before t; false: before the request
-            if (k.before >= back) nhv_load8(o, src - (size_t)back * p.qkv_stride + c * 8);
-            else if (k.has_past) nhv_load8(o, k.state + (size_t)(p.K - 1 + k.before - back) * C + at);
-            else return false;
-            return true;
-          };
-          if constexpr (TAPS > 0) {
-            float in[TAPS][8];
-            bool there[TAPS];
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) there[j] = j >= TAPS - p.K && past(in[j], TAPS - 1 - j);
+        for (int j = 0; j < TAPS; ++j) {
+          const int back = X - j;
+          if (j < skip) continue;
+          float o[8], w[8];
+          if (k.before >= back) raw_get(o, in[i + j]);
+          else if (k.has_past) nhv_load8(o, k.state + (size_t)(p.K - 1 + k.before - back) * C + at);
+          else continue;
+          raw_get(w, tap[j]);
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j)
-              if (there[j])
-#pragma unroll
-                for (int e = 0; e < 8; ++e) v[e] = fmaf(tap[j][e], in[j][e], v[e]);
-          } else {
-            for (int j = 0; j < p.K; ++j) {
-              float in[8], w[8];
-              if (!past(in, p.K - 1 - j)) continue;
-              nhv_load8(w, p.taps + (size_t)j * C + at);
-#pragma unroll
-              for (int e = 0; e < 8; ++e) v[e] = fmaf(w[e], in[e], v[e]);
+          for (int e = 0; e < 8; ++e) v[e] = fmaf(w[e], o[e], v[e]);
+        }
+        if (k.single && k.state && p.K > 1) {               // the only reader of these channels of this state
+          float o[8];
+          for (int j = 0; j + 2 < p.K; ++j) {
+            if (k.has_past) {
+              nhv_load8(o, k.state + (size_t)(j + 1) * C + at);
+              nhv_store8(k.state + (size_t)j * C + at, o);
+            } else {
+              nhv_store8(k.state + (size_t)j * C + at, zero);
             }
           }
-          if (k.single && k.state && p.K > 1) {             // the only reader of these channels of this state
-            float in[8];
-            for (int j = 0; j + 2 < p.K; ++j) {
-              if (k.has_past) {
-                nhv_load8(in, k.state + (size_t)(j + 1) * C + at);
-                nhv_store8(k.state + (size_t)j * C + at, in);
-              } else {
-                nhv_store8(k.state + (size_t)j * C + at, zero);
-              }
-            }
-            nhv_load8(in, src + c * 8);
-            nhv_store8(k.state + (size_t)(p.K - 2) * C + at, in);
-          }
-        } else {
-          nhv_load8(v, src + c * 8);
+          raw_get(o, in[i + X]);
+          nhv_store8(k.state + (size_t)(p.K - 2) * C + at, o);
         }
         if (u.dst_v) nhv_store8(u.dst_v + c * 8, v);
       }
       if (live && kind == 1 && u.dst_v)
         for (int y = CH + c; y < p.row / 8; y += L) nhv_store8(u.dst_v + y * 8, zero);
-      if (p.eps >= 0.f) {
-        float ss = 0.f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
-#pragma unroll
-        for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        const float r = 1.0f / sqrtf(ss / (float)p.dk + p.eps);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = v[e] * r * hw[e];
-      }
+      if (live && kind == 2 && u.dst)
+        for (int y = c; y < p.row / 8; y += L) {
+          float val[8];
+          if (y < p.dv / 8) {
+            nhv_load8(val, p.qkv + (size_t)(t0 + i) * p.qkv_stride + u.col + y * 8);
+            nhv_store8(u.dst + y * 8, val);
+          } else {
+            nhv_store8(u.dst + y * 8, zero);
+          }
+        }
       const float* cs = heads_angles(p, k.pos);
-      if (cs) {
-        float co[8], si[8];
-        if (mine && turns) {
-          nhv_load8(co, cs + i0);
-          nhv_load8(si, cs + half + i0);
-        }
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float other = __shfl_sync(0xffffffffu, v[e], partner, L);
-          if (mine && turns) v[e] = first ? v[e] * co[e] - other * si[e] : v[e] * co[e] + other * si[e];
-        }
+      float co[8], si[8];
+      if (cs && mine && lane.turns) {
+        nhv_load8(co, cs + lane.i0);
+        nhv_load8(si, cs + (p.rotary_dim >> 1) + lane.i0);
       }
-      if (!live || kind == 2 || !u.dst) continue;           // no exchange from here on
-      const int from = u.map * CH;
-      if (mine) {
-        if (kind == 0) {
-          const float f = temp[i];
-#pragma unroll
-          for (int e = 0; e < 8; ++e) v[e] *= f;
-        }
-        nhv_store8(u.dst + (from + c) * 8, v);
-      }
-      if (kind == 0) {
-        for (int y = c; y < p.q_head / 8; y += L)
-          if (y < from || y >= from + CH) nhv_store8(u.dst + y * 8, zero);
-      } else if (u.map == p.maps - 1) {
-        for (int y = p.maps * CH + c; y < p.row / 8; y += L) nhv_store8(u.dst + y * 8, zero);
-      }
+      heads_finish<T, L>(p, v, u, live, mine, lane, hw, cs != nullptr, co, si, temps[i]);
     }
   }
 }
@@ -384,27 +465,28 @@ static int heads_store_launch(HeadsStore<T> p, bool portions, cudaStream_t strea
   const bool vec = p.dk % 8 == 0 && p.dk <= 256 && p.q_head % 8 == 0 && p.qkv_stride % 8 == 0 && p.q_out_stride % 8 == 0 &&
                    (!p.cos_sin || (half % 8 == 0 && ok16(p.cos_sin))) &&
                    (!p.kv_pages || (p.row % 8 == 0 && (p.v_from_k || p.dv % 8 == 0))) &&
-                   (!p.taps || p.K < 2 || p.state_stride % 4 == 0) && ok16(p.qkv) && ok16(p.q_out) && ok16(p.kv_pages) &&
+                   (!p.taps || (p.K <= HS_TAPS && (p.K < 2 || p.state_stride % 4 == 0))) && ok16(p.qkv) && ok16(p.q_out) && ok16(p.kv_pages) &&
                    ok16(p.q_weight) && ok16(p.k_weight) && ok16(p.taps) && ok16(p.state);
   if (vec) {
     const int ch = p.dk / 8, L = ch <= 4 ? 4 : ch <= 8 ? 8 : ch <= 16 ? 16 : 32;
-    // long steps: several tokens a block, so that a unit's taps and weights are read once for them; short steps: a block
-    // per share of a token's units
-    const int tokens = p.n_tokens >= 2048 ? HS_TOKENS : 1;
-    const int blocks = (p.n_tokens + tokens - 1) / tokens, passes = (p.units + HS_THREADS / L - 1) / (HS_THREADS / L);
-    const dim3 grid(blocks, blocks >= 592 ? 1 : passes);
-#define GO(L, TAPS) nhv_launch(heads_store_vec_kernel<T, L, TAPS>, grid, HS_THREADS, 0, stream, p, tokens)
-#define PICK(L)                                  \
-  do {                                           \
-    if (!p.taps) GO(L, 0);                       \
-    else if (p.K <= HS_TAPS) GO(L, HS_TAPS);     \
-    else GO(L, -1);                              \
+    // short steps: a block per share of a token's units; long steps: a block for all of them, with a filter for several tokens
+    const int passes = (p.units + HS_THREADS / L - 1) / (HS_THREADS / L);
+    const bool many = p.n_tokens >= 2048;
+#define GO(L)                                                                                                        \
+  do {                                                                                                               \
+    if (!p.taps)                                                                                                     \
+      nhv_launch(heads_store_vec_kernel<T, L>, dim3(p.n_tokens, p.n_tokens >= 592 ? 1 : passes), HS_THREADS, 0, stream, p); \
+    else if (many)                                                                                                   \
+      nhv_launch(heads_filter_vec_kernel<T, L, HS_TAPS, HS_TOKENS>, dim3((p.n_tokens + HS_TOKENS - 1) / HS_TOKENS),  \
+                 HS_THREADS, 0, stream, p);                                                                          \
+    else                                                                                                             \
+      nhv_launch(heads_filter_vec_kernel<T, L, HS_TAPS, 1>, dim3(p.n_tokens, p.n_tokens >= 592 ? 1 : passes), HS_THREADS, 0, \
+                 stream, p);                                                                                         \
   } while (0)
-    if (L == 4) PICK(4);
-    else if (L == 8) PICK(8);
-    else if (L == 16) PICK(16);
-    else PICK(32);
-#undef PICK
+    if (L == 4) GO(4);
+    else if (L == 8) GO(8);
+    else if (L == 16) GO(16);
+    else GO(32);
 #undef GO
   } else {
     const size_t smem = (size_t)HS_WARPS * p.dk * sizeof(float);
