@@ -748,12 +748,12 @@ def kilisun_config(width: int, heads: int, ff: int, layers: int) -> dict:
     second differential layer that reads the first one's keys, and attention over all keys again.  The first layer of
     every four has the dense feed-forward ``ff``; the others a mixture of 16 experts in 4 groups of which 2 are kept, a
     token uses 4, and a shared expert: together as wide as ``ff`` (4 * 2/11 + 3/11 of it)."""
-    moe = dict(kind="moe", router=dict(experts=16, top=4, groups=dict(count=4, keep=2), scale=2.0),
+    moe = dict(kind="moe", router=dict(experts=16, top=4, groups=dict(count=4, keep=2), scale=1.5),
                expert=dict(ff=ff * 2 // 11, limit=7.0), shared=dict(ff=ff * 3 // 11, limit=7.0))
     kv = max(heads // 4, 1)
-    maps = dict(heads=heads, kv_heads=kv, dim=64, vdim=128, scale=64 ** -0.5, diff=0.6, softcap=30.0,
+    maps = dict(heads=heads, kv_heads=kv, dim=64, vdim=128, scale=64 ** -0.5, diff=0.7, softcap=30.0,
                 rot=dict(base=500000.0, dims=64), mask=dict(size=1024))
-    full = dict(heads=heads, kv_heads=kv, dim=128, vdim=128, scale=128 ** -0.5, conv=3, q_temp=dict(coef=0.3, every=1024))
+    full = dict(heads=heads, kv_heads=kv, dim=128, vdim=128, scale=128 ** -0.5, conv=3, q_temp=dict(coef=0.2, every=1024))
     out = []
     for i in range(layers):
         mixer = full if i % 2 else (dict(maps, kv_from=i - 2) if i % 4 == 2 else maps)
